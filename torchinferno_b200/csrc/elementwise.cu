@@ -16,43 +16,69 @@
 namespace tib {
 
 // ---------------------------------------------------------------- embedding
+// out = table[id] * scale (+ a row of a second table of the same type, chosen by position).
+struct EmbeddingArgs {
+  const int* ids; int hidden, vocab;
+  float scale;
+  const int* positions; const void* position_table; int max_positions;      // or null
+};
+
 template <typename T>
-__global__ void embedding_kernel(const int* __restrict__ ids, const T* __restrict__ table,
-                                 float* __restrict__ out, int hidden, int vocab) {
+__global__ void embedding_kernel(const T* __restrict__ table, float* __restrict__ out, EmbeddingArgs a) {
   pdl_wait();
   pdl_trigger();
   const int row = blockIdx.x;
-  const int id = ids[row];
-  float* dst = out + (size_t)row * hidden;
-  if (id < 0 || id >= vocab) {  // an id outside the table must show, not alias a row
-    for (int c = threadIdx.x; c < hidden; c += blockDim.x) dst[c] = __int_as_float(0x7fc00000);
+  const int id = a.ids[row], pos = a.positions ? a.positions[row] : 0;
+  float* dst = out + (size_t)row * a.hidden;
+  // an id or a position outside its table must show, not alias a row
+  if (id < 0 || id >= a.vocab || (a.positions && (pos < 0 || pos >= a.max_positions))) {
+    for (int c = threadIdx.x; c < a.hidden; c += blockDim.x) dst[c] = __int_as_float(0x7fc00000);
     return;
   }
-  const T* src = table + (size_t)id * hidden;
-  for (int c = threadIdx.x; c < hidden; c += blockDim.x) dst[c] = to_f32(src[c]);
+  const T* src = table + (size_t)id * a.hidden;
+  const T* at = a.positions ? reinterpret_cast<const T*>(a.position_table) + (size_t)pos * a.hidden : nullptr;
+  for (int c = threadIdx.x; c < a.hidden; c += blockDim.x) {
+    float v = to_f32(src[c]) * a.scale;
+    if (at) v += to_f32(at[c]);
+    dst[c] = v;
+  }
 }
 
 // bf16 table, width a multiple of 8: eight elements a thread and pass (one 16-byte load, two 16-byte stores), so that
 // a row of a few thousand columns is one or two passes of a block and not sixteen (7.6 -> about 2 us for the eight
 // rows of a decode step, which is all latency).
-__global__ void embedding_bf16x8_kernel(const int* __restrict__ ids, const __nv_bfloat16* __restrict__ table,
-                                        float* __restrict__ out, int hidden, int vocab) {
+__global__ void embedding_bf16x8_kernel(const __nv_bfloat16* __restrict__ table, float* __restrict__ out, EmbeddingArgs a) {
   pdl_wait();
   pdl_trigger();
   const int row = blockIdx.x;
-  const int id = ids[row];
-  float* dst = out + (size_t)row * hidden;
-  const bool known = id >= 0 && id < vocab;        // an id outside the table must show, not alias a row
-  const __nv_bfloat16* src = table + (size_t)(known ? id : 0) * hidden;
+  const int id = a.ids[row], pos = a.positions ? a.positions[row] : 0;
+  float* dst = out + (size_t)row * a.hidden;
+  // (an id or a position outside its table must show, not alias a row)
+  const bool known = id >= 0 && id < a.vocab && (!a.positions || (pos >= 0 && pos < a.max_positions));
+  const __nv_bfloat16* src = table + (size_t)(known ? id : 0) * a.hidden;
+  const __nv_bfloat16* at = reinterpret_cast<const __nv_bfloat16*>(a.position_table) + (size_t)(known ? pos : 0) * a.hidden;
   const float nan = __int_as_float(0x7fc00000);
-  for (int c = threadIdx.x * 8; c < hidden; c += blockDim.x * 8) {
+  for (int c = threadIdx.x * 8; c < a.hidden; c += blockDim.x * 8) {
     float4 lo = make_float4(nan, nan, nan, nan), hi = lo;
     if (known) {
       const uint4 raw = *reinterpret_cast<const uint4*>(src + c);
+      uint4 add = make_uint4(0, 0, 0, 0);
+      if (a.positions) add = *reinterpret_cast<const uint4*>(at + c);
       const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
-      const float2 a = bf16x2_floats(p[0]), b = bf16x2_floats(p[1]), e = bf16x2_floats(p[2]), f = bf16x2_floats(p[3]);
-      lo = make_float4(a.x, a.y, b.x, b.y);
-      hi = make_float4(e.x, e.y, f.x, f.y);
+      const __nv_bfloat162* q = reinterpret_cast<const __nv_bfloat162*>(&add);
+      float v[8];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float2 f = bf16x2_floats(p[i]), g = bf16x2_floats(q[i]);
+        v[2 * i] = f.x * a.scale;
+        v[2 * i + 1] = f.y * a.scale;
+        if (a.positions) {
+          v[2 * i] += g.x;
+          v[2 * i + 1] += g.y;
+        }
+      }
+      lo = make_float4(v[0], v[1], v[2], v[3]);
+      hi = make_float4(v[4], v[5], v[6], v[7]);
     }
     *reinterpret_cast<float4*>(dst + c) = lo;
     *reinterpret_cast<float4*>(dst + c + 4) = hi;
@@ -268,18 +294,23 @@ static inline int norm_threads(int hidden) {
 
 using namespace tib;
 
-TIB_API int tib_embedding(const int* ids, const void* table, float* out, int n_tokens, int hidden,
-                          int vocab, int dtype, cudaStream_t stream) {
+// out[t] = table[ids[t]] * scale, plus position_table[positions[t]] where positions is not null ([max_positions, hidden] of the
+// same dtype).
+TIB_API int tib_embedding(const int* ids, const void* table, float* out, int n_tokens, int hidden, int vocab, float scale,
+                          const int* positions, const void* position_table, int max_positions, int dtype, cudaStream_t stream) {
   if (n_tokens == 0) return TIB_OK;
-  if (!ids || !table || !out || n_tokens < 0 || hidden < 1 || vocab < 1) return TIB_E_ARG;
+  if (!ids || !table || !out || n_tokens < 0 || hidden < 1 || vocab < 1 || (positions && (!position_table || max_positions < 1))) return TIB_E_ARG;
+  EmbeddingArgs a;
+  a.ids = ids; a.hidden = hidden; a.vocab = vocab; a.scale = scale; a.positions = positions; a.position_table = position_table;
+  a.max_positions = max_positions;
   const int threads = hidden >= 1024 ? 256 : 128;
   if (dtype == TIB_F32)
-    TIB_LAUNCH_DEPENDENT(embedding_kernel<float>, n_tokens, threads, 0, stream, ids, (const float*)table, out, hidden, vocab);
-  else if (dtype == TIB_BF16 && hidden % 8 == 0 && (((uintptr_t)table | (uintptr_t)out) & 15) == 0)
-    TIB_LAUNCH_DEPENDENT(embedding_bf16x8_kernel, n_tokens, hidden >= 4096 ? 512 : hidden >= 1024 ? 128 : 64, 0, stream, ids,
-                         (const __nv_bfloat16*)table, out, hidden, vocab);
+    TIB_LAUNCH_DEPENDENT(embedding_kernel<float>, n_tokens, threads, 0, stream, (const float*)table, out, a);
+  else if (dtype == TIB_BF16 && hidden % 8 == 0 && (((uintptr_t)table | (uintptr_t)out | (uintptr_t)position_table) & 15) == 0)
+    TIB_LAUNCH_DEPENDENT(embedding_bf16x8_kernel, n_tokens, hidden >= 4096 ? 512 : hidden >= 1024 ? 128 : 64, 0, stream,
+                         (const __nv_bfloat16*)table, out, a);
   else if (dtype == TIB_BF16)
-    TIB_LAUNCH_DEPENDENT(embedding_kernel<__nv_bfloat16>, n_tokens, threads, 0, stream, ids, (const __nv_bfloat16*)table, out, hidden, vocab);
+    TIB_LAUNCH_DEPENDENT(embedding_kernel<__nv_bfloat16>, n_tokens, threads, 0, stream, (const __nv_bfloat16*)table, out, a);
   else
     return TIB_E_DTYPE;
   TIB_LAUNCH_CHECK();

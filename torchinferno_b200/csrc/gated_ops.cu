@@ -133,11 +133,17 @@ __global__ void pair_rows_kernel(const float* __restrict__ x, const float* __res
 }
 
 // x[t] += v (one fp32 vector for every row)
-__global__ void add_vector_kernel(float* __restrict__ x, const float* __restrict__ v, int width) {
+// x[t] += v, after x[t] += delta[t] where delta is not null
+__global__ void add_vector_kernel(float* __restrict__ x, const void* __restrict__ delta, int delta_dtype, int64_t ldd,
+                                  const float* __restrict__ v, int width) {
   pdl_wait();
   pdl_trigger();
   const size_t row = blockIdx.x;
-  for (int c = threadIdx.x; c < width; c += blockDim.x) x[row * width + c] += v[c];
+  for (int c = threadIdx.x; c < width; c += blockDim.x) {
+    float h = x[row * width + c];
+    if (delta) h += load_any(delta, delta_dtype, row * ldd + c);
+    x[row * width + c] = h + v[c];
+  }
 }
 
 static inline int row_threads(int width) { return width >= 1024 ? 256 : (width >= 256 ? 128 : 64); }
@@ -245,9 +251,11 @@ TIB_API int tib_pair_rows(const float* x, const float* y, void* out, int out_dty
   return TIB_OK;
 }
 
-TIB_API int tib_add_vector(float* x, const float* v, int rows, int width, cudaStream_t stream) {
+TIB_API int tib_add_vector(float* x, const void* delta, int delta_dtype, int64_t ldd, const float* v, int rows, int width,
+                           cudaStream_t stream) {
   if (rows == 0 || width == 0) return TIB_OK;
   if (!x || !v || rows < 0 || width < 0) return TIB_E_ARG;
-  TIB_LAUNCH_DEPENDENT(add_vector_kernel, rows, row_threads(width), 0, stream, x, v, width);
+  if (delta && !known(delta_dtype)) return TIB_E_DTYPE;
+  TIB_LAUNCH_DEPENDENT(add_vector_kernel, rows, row_threads(width), 0, stream, x, delta, delta_dtype, ldd, v, width);
   return TIB_OK;
 }

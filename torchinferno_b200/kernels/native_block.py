@@ -61,6 +61,8 @@ def block_weights(block) -> BlockWeights | None:
     from torchinferno_b200.parts.norm import RMSNorm
     from torchinferno_b200.parts.rope import NoPositionEncoding, RotaryEncoding
     mixer, ffn, n1, n2 = block.mixer, block.feed_forward, block.mixer_norm, block.feed_forward_norm
+    if block.mixer_input is not None or block.feed_forward_input is not None:
+        return None
     if block.dtype != torch.bfloat16 or block.device.type != "cuda" or gemm.get_backend() == "tcgen05":
         return None
     if type(mixer) is not GQAAttention or type(ffn) is not SwiGLUFeedForward or type(n1) is not RMSNorm or type(n2) is not RMSNorm:

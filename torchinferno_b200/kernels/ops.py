@@ -127,21 +127,33 @@ def lib() -> ctypes.CDLL:
                    "tib_qk_norm_append", "tib_sigmoid_attention", "tib_sigmoid_attention_takes_mma", "tib_gated_recurrence",
                    "tib_softcap_f32", "tib_short_conv", "tib_ssd_scan", "tib_ssd_scan_max_state", "tib_ssd_scan_run", "tib_gated_group_norm",
                    "tib_rotary_kv_append", "tib_pool_blocks", "tib_pooled_window_attention", "tib_hyper_step",
-                   "tib_pooled_window_attention_splits", "tib_pooled_window_attention_part_floats"):
+                   "tib_pooled_window_attention_splits", "tib_pooled_window_attention_part_floats",
+                   "tib_input_conv", "tib_norm_conv_step", "tib_row_norm_append", "tib_talking_heads_attention",
+                   "tib_talking_heads_takes_mma", "tib_talking_heads_takes_step", "tib_talking_heads_key_span",
+                   "tib_talking_heads_tiles_per_part"):
             getattr(library, fn).restype = c_int
         _signatures_set = True
     return library
 
 
 # ---------------------------------------------------------------------------
-def embedding(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-    """out[t] = float(table[ids[t]]): the residual stream starts in 32-bit."""
+def embedding(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, *, scale: float = 1.0,
+              positions: torch.Tensor | None = None, position_table: torch.Tensor | None = None) -> torch.Tensor:
+    """out[t] = float(table[ids[t]]) * scale (+ float(position_table[positions[t]])): the residual stream starts in 32-bit."""
     _need(ids, "ids", torch.int32), _need(table, "table"), _need(out, "out", torch.float32)
     n, (vocab, hidden) = ids.numel(), table.shape
     if out.shape != (n, hidden):
         raise KernelError(f"embedding: out is {tuple(out.shape)}, wanted {(n, hidden)}")
-    _check("embedding", lib().tib_embedding(_ptr(ids), _ptr(table), _ptr(out), c_int(n), c_int(hidden),
-                                            c_int(vocab), c_int(_code(table.dtype)), _stream()))
+    if position_table is not None:
+        if positions is None:
+            raise KernelError("embedding: a table of positions needs the tokens' positions")
+        _need(position_table, "position_table", table.dtype), _need(positions, "positions", torch.int32)
+        if position_table.dim() != 2 or position_table.shape[1] != hidden or positions.numel() != n:
+            raise KernelError("embedding: the table of positions does not fit")
+    _check("embedding", lib().tib_embedding(
+        _ptr(ids), _ptr(table), _ptr(out), c_int(n), c_int(hidden), c_int(vocab), c_float(scale),
+        _ptr(positions if position_table is not None else None), _ptr(position_table),
+        c_int(position_table.shape[0] if position_table is not None else 0), c_int(_code(table.dtype)), _stream()))
     return out
 
 
@@ -817,12 +829,18 @@ def pair_rows(x: torch.Tensor, y: torch.Tensor, out: torch.Tensor) -> torch.Tens
     return out
 
 
-def add_vector(x: torch.Tensor, v: torch.Tensor) -> torch.Tensor:
-    """x[t] += v for every row (fp32)."""
+def add_vector(x: torch.Tensor, v: torch.Tensor, delta: torch.Tensor | None = None) -> torch.Tensor:
+    """x[t] += v for every row, after x[t] += delta[t] when ``delta`` is given (fp32)."""
     _need(x, "x", torch.float32), _need(v, "v", torch.float32)
     if v.numel() != x.shape[1]:
         raise KernelError("add_vector: the vector has the wrong length")
-    _check("add_vector", lib().tib_add_vector(_ptr(x), _ptr(v), c_int(x.shape[0]), c_int(x.shape[1]), _stream()))
+    if delta is not None:
+        _rows_of(delta, "delta", x.shape[1])
+        if delta.shape[0] != x.shape[0]:
+            raise KernelError("add_vector: delta does not fit")
+    _check("add_vector", lib().tib_add_vector(
+        _ptr(x), _ptr(delta), c_int(_code(delta.dtype) if delta is not None else 0),
+        c_int64(delta.stride(0) if delta is not None else 0), _ptr(v), c_int(x.shape[0]), c_int(x.shape[1]), _stream()))
     return x
 
 
@@ -1496,4 +1514,175 @@ def hyper_step(streams: torch.Tensor, *, y: torch.Tensor | None = None, mix: tor
         c_int(_code(y.dtype) if y is not None else 0), c_int64(y.stride(0) if y is not None else 0), _ptr(mix),
         _ptr(out_weights), _ptr(in_weights), _ptr(rows), c_int(norm), c_float(alpha), _ptr(weight), _ptr(bias), _ptr(out),
         c_int(_code(out.dtype) if out is not None else 0), _stream()))
+    return out
+
+
+# ---------------------------------------------------------------------------
+# A short causal convolution added to a sublayer's input (csrc/input_conv.cu).
+def _conv_state(state: torch.Tensor | None, state_off: int, taps: int, width: int, name: str) -> int:
+    if taps == 1:
+        return 0
+    if state is None:
+        raise KernelError(f"{name}: a convolution of more than one tap carries rows in a state")
+    _need(state, "state", torch.float32)
+    if state.dim() != 2 or state_off < 0 or state_off + (taps - 1) * width > state.shape[1]:
+        raise KernelError(f"{name}: the state does not hold the carried rows")
+    return state.stride(0)
+
+
+def input_conv(x: torch.Tensor, out: torch.Tensor, weight: torch.Tensor, state: torch.Tensor | None, state_off: int,
+               q_start: torch.Tensor, slots: torch.Tensor, n_entries: int, max_q_len: int) -> torch.Tensor:
+    """out[t] = x[t] + sum_j weight[j] * x[t - taps + 1 + j] per channel, causal within each entry of the ragged batch;
+    ``weight``: [taps, width] fp32.  The taps - 1 rows before an entry's first token come from ``state[slot, state_off:]``
+    (laid out [taps - 1, width]), where the kernel then leaves the entry's last taps - 1 rows."""
+    _need(x, "x"), _need(out, "out", x.dtype), _need(weight, "weight", torch.float32)
+    _need(q_start, "q_start", torch.int32), _need(slots, "slots", torch.int32)
+    taps, width = weight.shape
+    if x.dim() != 2 or x.shape[1] != width or out.shape != x.shape or out.data_ptr() == x.data_ptr():
+        raise KernelError("input_conv: x and out are two arrays of rows as wide as the weight")
+    if q_start.numel() < n_entries + 1 or slots.numel() < n_entries:
+        raise KernelError("input_conv: entry arrays are shorter than n_entries")
+    stride = _conv_state(state, state_off, taps, width, "input_conv")
+    _check("input_conv", lib().tib_input_conv(
+        _ptr(x), _ptr(out), _ptr(weight), _ptr(state), c_int64(stride), c_int64(state_off), _ptr(q_start), _ptr(slots),
+        c_int(n_entries), c_int(max_q_len), c_int(width), c_int(taps), c_int(_code(x.dtype)), _stream()))
+    return out
+
+
+def norm_conv_step(delta: torch.Tensor | None, residual: torch.Tensor, norm_weight: torch.Tensor, eps: float, weight: torch.Tensor,
+                   state: torch.Tensor | None, state_off: int, slots: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """For a step of single tokens (row i in slot ``slots[i]``), in one launch: residual += delta (when given), h = RMS norm
+    of the new rows times ``norm_weight``, out = h + the convolution of :func:`input_conv`, carried rows moved on."""
+    _need(residual, "residual", torch.float32), _need(norm_weight, "norm_weight", torch.float32), _need(weight, "weight", torch.float32)
+    _need(out, "out"), _need(slots, "slots", torch.int32)
+    n, width = residual.shape
+    taps = weight.shape[0]
+    if weight.shape[1] != width or norm_weight.numel() != width or out.shape != (n, width) or slots.numel() < n:
+        raise KernelError("norm_conv_step: shapes do not fit")
+    if delta is not None:
+        _need(delta, "delta", out.dtype)
+        if delta.shape != (n, width):
+            raise KernelError("norm_conv_step: delta does not fit")
+    stride = _conv_state(state, state_off, taps, width, "norm_conv_step")
+    _check("norm_conv_step", lib().tib_norm_conv_step(
+        _ptr(delta), _ptr(residual), _ptr(norm_weight), c_float(eps), _ptr(weight), _ptr(state), c_int64(stride),
+        c_int64(state_off), _ptr(slots), _ptr(out), c_int(n), c_int(width), c_int(taps), c_int(_code(out.dtype)), _stream()))
+    return out
+
+
+# ---------------------------------------------------------------------------
+# Attention whose softmax weights are mixed across the heads (csrc/talking_heads.cu).
+def row_norm_append(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_out: torch.Tensor, keys: torch.Tensor,
+                    values: torch.Tensor, positions: torch.Tensor, token_slot: torch.Tensor, block_table: torch.Tensor, heads: int,
+                    kv_heads: int, dim: int, vdim: int, *, eps: float = 1e-6, q_bias: torch.Tensor | None = None,
+                    k_bias: torch.Tensor | None = None, v_bias: torch.Tensor | None = None, q_weight: torch.Tensor | None = None,
+                    k_weight: torch.Tensor | None = None, error_word: torch.Tensor | None = None) -> torch.Tensor:
+    """Add the biases to the q, k and v columns of the fused projection ``proj``, divide the whole q row and the whole k row
+    (all heads at once) by their root mean square and multiply them by a weight per element (weights None: not normed), write
+    q to ``q_out`` and k, v into their pages."""
+    _rows_of(proj, "proj"), _need(q_out, "q_out", proj.dtype), _need(positions, "positions", torch.int32)
+    _need(token_slot, "token_slot", torch.int32), _need(block_table, "block_table", torch.int32)
+    n = proj.shape[0]
+    if q_out.shape != (n, heads * dim) or keys.dtype != proj.dtype:
+        raise KernelError("row_norm_append: shapes or types do not fit")
+    if max(q_off + heads * dim, k_off + kv_heads * dim, v_off + kv_heads * vdim) > proj.shape[1]:
+        raise KernelError("row_norm_append: the projection is narrower than its parts")
+    for t, width in ((q_bias, heads * dim), (k_bias, kv_heads * dim), (v_bias, kv_heads * vdim), (q_weight, heads * dim),
+                     (k_weight, kv_heads * dim)):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != width or not t.is_contiguous()):
+            raise KernelError("row_norm_append: a bias or a weight does not fit")
+    num_pages, page_size, page_stride = _pages(keys, values, kv_heads, dim, vdim, "row_norm_append")
+    _check("row_norm_append", lib().tib_row_norm_append(
+        _ptr(proj), c_int64(proj.stride(0)), c_int(q_off), c_int(k_off), c_int(v_off), _ptr(q_bias), _ptr(k_bias), _ptr(v_bias),
+        _ptr(q_weight), _ptr(k_weight), c_float(eps), _ptr(q_out), _ptr(keys), _ptr(values), _ptr(positions), _ptr(token_slot),
+        _ptr(block_table), c_int(block_table.stride(0)), c_int(n), c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim),
+        c_int(page_size), c_int64(page_stride), c_int(num_pages), _ptr(error_word), c_int(_code(proj.dtype)), _stream()))
+    return q_out
+
+
+# Bytes of scratch the three kernels of a portion pass their words through: what stays in the L2 between them.
+TALKING_HEADS_SCRATCH = 64 << 20
+
+
+def talking_heads_attention(q: torch.Tensor, out: torch.Tensor, q_start: torch.Tensor, kv_start: torch.Tensor, slots: torch.Tensor,
+                            positions: torch.Tensor, keys: torch.Tensor, values: torch.Tensor, block_table: torch.Tensor,
+                            n_entries: int, max_q_len: int, heads: int, kv_heads: int, *, window: int, scale: float,
+                            talk: torch.Tensor, talk_hi: torch.Tensor | None = None, talk_lo: torch.Tensor | None = None,
+                            softcap: float = 0.0, bias: torch.Tensor | None = None, gate: torch.Tensor | None = None,
+                            max_kv_len: int = 0, error_word: torch.Tensor | None = None, force_simt: bool = False,
+                            force_portions: bool = False, tiles_per_part: int | None = None,
+                            scratch_bytes: int | None = None) -> torch.Tensor:
+    """Per head h, out[i] = sigmoid(gate[i]) * sum_j (sum_g talk[h, g] w_g(i, j)) v_j over the tokens j with 0 <= i - j <
+    ``window``; w_g(i, .) = softmax of cap(q_i . k_j * scale) + bias[g, min(i - j, span - 1)], cap(s) = softcap * tanh(s /
+    softcap) (0: none).  ``talk``: [heads, heads] fp32; ``talk_hi`` / ``talk_lo``: the same as two bf16 terms, padded with zeros
+    to multiples of 16 (``talk_lo`` None: the first term is exact).  ``max_kv_len``: a bound on the longest context.
+
+    bfloat16 with head sizes in steps of 8 up to 128 and at most 64 heads runs on the tensor cores: a step of single tokens
+    with up to 16 query heads a key head in two kernels over parts of ``tiles_per_part`` tiles of 64 keys, any other step in
+    three kernels over ranges of tokens whose scratch is at most ``scratch_bytes``.  Everything else (and ``force_simt``) runs
+    on the CUDA cores."""
+    _need(q, "q"), _need(out, "out", q.dtype), _need(talk, "talk", torch.float32)
+    for name, t in (("q_start", q_start), ("kv_start", kv_start), ("slots", slots), ("positions", positions)):
+        _need(t, name, torch.int32)
+    dim, vdim = keys.shape[3], values.shape[3]
+    n = q.shape[0]
+    if q.shape != (n, heads * dim) or out.shape != (n, heads * vdim) or keys.dtype != q.dtype or talk.shape != (heads, heads):
+        raise KernelError("talking_heads_attention: shapes or types do not fit")
+    if q_start.numel() < n_entries + 1 or kv_start.numel() < n_entries or slots.numel() < n_entries or positions.numel() < n:
+        raise KernelError("talking_heads_attention: an array of the batch is too short")
+    num_pages, page_size, page_stride = _pages(keys, values, kv_heads, dim, vdim, "talking_heads_attention")
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+        if bias.dim() != 2 or bias.shape[0] != heads or bias.shape[1] < 1:
+            raise KernelError("talking_heads_attention: bias must be [heads, span]")
+    ld_gate = 0
+    if gate is not None:
+        _rows_of(gate, "gate", heads * vdim)
+        ld_gate = gate.stride(0)
+
+    def call(form, first=0, last=0, scores=None, lse=None, key_span=0, part_ml=None, part_o=None, counters=None, tiles=0, parts=0):
+        _check("talking_heads_attention", lib().tib_talking_heads_attention(
+            _ptr(q), _ptr(out), _ptr(q_start), _ptr(kv_start), _ptr(slots), _ptr(positions), _ptr(keys), _ptr(values), _ptr(block_table),
+            c_int(block_table.stride(0)), c_int(page_size), c_int64(page_stride), c_int(num_pages), c_int(n_entries), c_int(max_q_len),
+            c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim), c_int(window), c_float(scale), c_float(softcap), _ptr(bias),
+            c_int(bias.shape[1] if bias is not None else 0), _ptr(talk), _ptr(talk_hi), _ptr(talk_lo), _ptr(gate),
+            c_int(_code(gate.dtype) if gate is not None else 0), c_int64(ld_gate), c_int(form), c_int(first), c_int(last),
+            _ptr(scores), _ptr(lse), c_int(key_span), _ptr(part_ml), _ptr(part_o), _ptr(counters), c_int(tiles), c_int(parts),
+            _ptr(error_word), c_int(_code(q.dtype)), _stream()))
+
+    if q.dtype != torch.bfloat16 or force_simt or not lib().tib_talking_heads_takes_mma(c_int(heads), c_int(dim), c_int(vdim)):
+        call(0)
+        return out
+    if max_kv_len < 1:
+        raise KernelError("talking_heads_attention: the tensor-core forms need a bound on the longest context")
+    key_span = int(lib().tib_talking_heads_key_span(c_int(window), c_int(max_kv_len)))
+    if (max_q_len == 1 and n == n_entries and not force_portions
+            and lib().tib_talking_heads_takes_step(c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim))):
+        tiles = tiles_per_part or int(lib().tib_talking_heads_tiles_per_part(c_int(n_entries), c_int(kv_heads), c_int(key_span)))
+        parts = -(-key_span // (64 * tiles))
+        scores = torch.empty((n, heads, key_span), dtype=torch.float32, device=q.device)
+        part_ml = torch.empty((n, parts, heads, 2), dtype=torch.float32, device=q.device)
+        part_o = torch.empty((n, parts, heads, 128), dtype=torch.float32, device=q.device)
+        counters = _split_counters(q.device, n_entries * kv_heads)
+        if counters is None:
+            tiles, parts = key_span // 64, 1          # (more rows than counters: no context is shared out)
+            counters = _split_counters(q.device, 1)
+        count_launches(1)
+        call(2, scores=scores, key_span=key_span, part_ml=part_ml, part_o=part_o, counters=counters, tiles=tiles, parts=parts)
+        return out
+    if talk_hi is None:
+        raise KernelError("talking_heads_attention: the tensor-core form needs talk_hi")
+    padded = 16 if heads <= 16 else 32 if heads <= 32 else 64
+    for t in (talk_hi, talk_lo):
+        if t is not None and (t.dtype != torch.bfloat16 or tuple(t.shape) != (padded, padded) or not t.is_contiguous()):
+            raise KernelError(f"talking_heads_attention: talk_hi and talk_lo must be [{padded}, {padded}] bf16")
+    row = heads * key_span * 4
+    chunk = max(64, (TALKING_HEADS_SCRATCH if scratch_bytes is None else scratch_bytes) // row)
+    pieces = -(-n // chunk)
+    chunk = -(-n // pieces)                           # (equal ranges)
+    scores = torch.empty((chunk, heads, key_span), dtype=torch.float32, device=q.device)
+    lse = torch.empty((chunk, heads), dtype=torch.float32, device=q.device)
+    for first in range(0, n, chunk):
+        count_launches(2)
+        call(1, first=first, last=min(n, first + chunk), scores=scores, lse=lse, key_span=key_span)
     return out

@@ -34,6 +34,7 @@ class CausalLM:
         self.stages = [build_part("stream_stage", stage, dtype=dtype, device=self.device) for stage in spec.stages]
         self.embedding: torch.Tensor | None = None
         self.head: torch.Tensor | None = None
+        self.position_table: torch.Tensor | None = None
 
     def _owned_parts(self):
         """(full name prefix, part) of every part that owns weights, blocks first."""
@@ -61,6 +62,9 @@ class CausalLM:
                 if ws.name in expected and tuple(expected[ws.name].shape) != tuple(ws.shape):
                     raise ValueError(f"{ws.name}: parts that share it declare shapes {expected[ws.name].shape} and {ws.shape}")
                 expected[ws.name] = ws
+        if spec.position_embedding_name is not None:
+            name = spec.position_embedding_name
+            expected[name] = WeightSpec(name, (spec.max_positions, spec.hidden_size), std=0.5)
         if spec.head_name is not None:
             expected[spec.head_name] = WeightSpec(
                 spec.head_name, (spec.vocab_size, spec.hidden_size), optional=spec.tie_head_to_embedding)
@@ -78,6 +82,8 @@ class CausalLM:
         spec = self.spec
         take = tensors.pop if consume else tensors.__getitem__
         self.embedding = take(spec.embedding_name)
+        if spec.position_embedding_name is not None:
+            self.position_table = take(spec.position_embedding_name).to(self.embedding.dtype)
         if spec.tie_head_to_embedding or spec.head_name is None:
             self.head = self.embedding
         elif spec.head_name in tensors:
@@ -140,12 +146,16 @@ class CausalLM:
         """Whether a decode step of this model may be captured in a CUDA graph (see ``Mixer.capturable``)."""
         parts = [block.mixer for block in self.blocks] + ([self.after_embedding] if self.after_embedding is not None else []) \
             + list(self.stages)
-        return all(getattr(part, "capturable", getattr(part, "state_spec", lambda: None)() is None) for part in parts)
+        return all(block.capturable for block in self.blocks) and \
+            all(getattr(part, "capturable", getattr(part, "state_spec", lambda: None)() is None) for part in parts)
 
     def state_requirements(self) -> list[StateSpec | None]:
-        """StateSpec of every layer call of the schedule (None where the mixer has none)."""
-        return [None if isinstance(call, StageCall) else self.blocks[call.layer].mixer.state_spec()
-                for call in self.spec.schedule]
+        """StateSpec of every layer call of the schedule (None where the mixer has none); if any block keeps state outside
+        its mixer, as many entries again for the blocks."""
+        calls = [None if isinstance(call, StageCall) else self.blocks[call.layer] for call in self.spec.schedule]
+        mixers = [None if block is None else block.mixer.state_spec() for block in calls]
+        blocks = [None if block is None else block.block_state_spec() for block in calls]
+        return mixers + blocks if any(spec is not None for spec in blocks) else mixers
 
     # ------------------------------------------------------------ forward
     def forward(self, batch, cache) -> torch.Tensor:
@@ -160,9 +170,8 @@ class CausalLM:
             residual = history[0]
         else:
             residual = torch.empty((n, self.spec.hidden_size), dtype=torch.float32, device=self.device)
-        ops.embedding(batch.token_ids, self.embedding, residual)
-        if self.spec.embedding_scale != 1.0:
-            ops.scale_(residual, self.spec.embedding_scale)
+        ops.embedding(batch.token_ids, self.embedding, residual, scale=self.spec.embedding_scale, positions=batch.positions,
+                      position_table=self.position_table)
         if depth:
             history[1].copy_(residual)
             residual = history[1]
@@ -188,7 +197,8 @@ class CausalLM:
                 b = cache.kv_binding(call.side_cache)
                 side = KVBinding(b.pool, b.block_table, b.page_size, b.window, True, b.keys, b.values)
             ctx = LayerContext(batch=batch, kv=kv, state=cache.state(index),
-                               error_word=cache.error_word, layer_index=index, side_kv=side)
+                               error_word=cache.error_word, layer_index=index, side_kv=side,
+                               block_state=cache.state(len(self.spec.schedule) + index))
             self.blocks[call.layer].forward(stream, ctx)
         if batch.n_logits == 0:
             return torch.empty((0, self.spec.vocab_size), dtype=torch.float32, device=self.device)

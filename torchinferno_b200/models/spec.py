@@ -55,6 +55,8 @@ class ModelSpec:
     logit_scale: float = 1.0                  # the head's output is multiplied by this
     keeps_embedding_output: bool = False      # stages read the embedding output (``ResidualStream.origin``)
     embedding_scale: float = 1.0              # the embedding output is multiplied by this
+    position_embedding_name: str | None = None   # tensor [max_positions, hidden]: row p is added to the (scaled) embedding
+                                              # output of the token at position p
     logit_softcap: float | None = None        # c > 0: logits <- c * tanh(logits / c), after ``logit_scale``
     history_depth: int = 0                    # > 0: the residual stream lives in a [depth, tokens, hidden] tensor whose
                                               # slice 0 keeps the embedding output and whose later slices keep what

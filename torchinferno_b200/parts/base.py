@@ -18,6 +18,7 @@ Interfaces
 ``FeedForward``    ``forward(x, ctx) -> y``
 ``Block``          ``forward(stream, ctx)`` on a :class:`ResidualStream`
 ``StreamStage``    ``forward(stream, ctx)`` between the embedding and the first block
+``InputStage``     ``state_floats()``, ``forward(stream, norm, ctx, state_off) -> rows``: what a sublayer of a block reads
 """
 from __future__ import annotations
 
@@ -108,6 +109,7 @@ class LayerContext:
     layer_index: int = 0
     call_arg: int = 0                   # the argument of a stage call of the schedule
     side_kv: KVBinding | None = None    # the second cache of a mixer that keeps one (``Mixer.side_cache_spec``)
+    block_state: torch.Tensor | None = None   # [slots, *StateSpec.shape] of the block itself (``Block.block_state_spec``)
 
 
 class ResidualStream:
@@ -279,6 +281,15 @@ class Block(Part):
         """(prefix relative to the block, part) for every part that owns weights."""
         raise NotImplementedError
 
+    def block_state_spec(self) -> StateSpec | None:
+        """Per-request state of the block outside its mixer (``ctx.block_state``): what its input stages carry, say."""
+        return None
+
+    @property
+    def capturable(self) -> bool:
+        """Whether the block outside its mixer only launches kernels (see ``Mixer.capturable``)."""
+        return True
+
 
 class StreamStage(Part):
     """Something done to the residual stream once, after the embedding and before the first block: a learned
@@ -288,8 +299,22 @@ class StreamStage(Part):
         raise NotImplementedError
 
 
+class InputStage(Part):
+    """Makes what a sublayer reads from the residual stream and the sublayer's norm, with a fixed number of fp32 values of
+    state per request if it looks back in time: ``ctx.block_state[slot, state_off : state_off + state_floats()]``, zeroed for
+    a new request."""
+    capturable = False      # True: the forward only launches kernels that read the batch through its device arrays
+
+    def state_floats(self) -> int:
+        return 0
+
+    def forward(self, stream: ResidualStream, norm: Norm, ctx: LayerContext, state_off: int) -> torch.Tensor:
+        """The rows the sublayer reads, in the stream's activation type; the stream's pending sum is settled on the way."""
+        raise NotImplementedError
+
+
 # ----------------------------------------------------------------- registry
-_KINDS = ("mixer", "feed_forward", "norm", "position", "block", "stream_stage")
+_KINDS = ("mixer", "feed_forward", "norm", "position", "block", "stream_stage", "input_stage")
 _REGISTRY: dict[str, dict[str, Callable[..., Part]]] = {kind: {} for kind in _KINDS}
 
 
@@ -327,6 +352,6 @@ def _ensure_builtin() -> None:
         return
     _loaded = True
     from torchinferno_b200.parts import (attention, biased_attention, block, gated_recurrence, hyper_block,  # noqa: F401
-                                         latent_attention, linear_attention, mlp, moe, norm, parallel_block,
+                                         input_stages, latent_attention, linear_attention, mlp, moe, norm, parallel_block,
                                          pooled_window_attention, rope, sandwich_block, sigmoid_attention, state_space,
-                                         stream_stages)
+                                         stream_stages, talking_heads_attention)

@@ -3,7 +3,9 @@
 y = x * rsqrt(mean(x^2) + eps) * w with the statistics, the product and the
 residual sum in fp32 (src/torchinferno/models/llama3/raw_ops.py:9-11,
 src/torchinferno/kernels/triton_ops.py:2044-2048, 2088-2096).  The weight
-multiplies after normalisation; there is no bias and no ``1 + w`` form.
+multiplies after normalisation; there is no bias.  ``weight_offset`` is added to
+the stored weight when it is bound (1 for checkpoints that store what the gain
+exceeds 1 by).
 """
 from __future__ import annotations
 
@@ -16,17 +18,20 @@ from torchinferno_b200.parts.base import Norm, WeightSpec, register_part
 
 
 class RMSNorm(Norm):
-    def __init__(self, *, width: int, eps: float, weight_name: str = "weight",
+    def __init__(self, *, width: int, eps: float, weight_name: str = "weight", weight_offset: float = 0.0,
                  dtype: torch.dtype, device: torch.device) -> None:
         super().__init__(dtype=dtype, device=device)
-        self.width, self.eps, self.weight_name = int(width), float(eps), weight_name
+        self.width, self.eps, self.weight_name, self.weight_offset = int(width), float(eps), weight_name, float(weight_offset)
         self.weight: torch.Tensor | None = None
 
     def weight_specs(self) -> list[WeightSpec]:
+        if self.weight_offset:
+            return [WeightSpec(self.weight_name, (self.width,), std=0.1, role="vector")]
         return [WeightSpec(self.weight_name, (self.width,), init="ones", role="vector")]
 
     def bind(self, weights: Mapping[str, torch.Tensor]) -> None:
-        self.weight = weights[self.weight_name].to(torch.float32).contiguous()
+        weight = weights[self.weight_name].to(torch.float32).contiguous()
+        self.weight = weight + self.weight_offset if self.weight_offset else weight
 
     def forward(self, residual, out, rows=None):
         return ops.add_rmsnorm(None, residual, self.weight, self.eps, out, rows)

@@ -6,6 +6,7 @@
                 the sublayers' sum (parts/parallel_block.py), and reads the residual itself, not a normed copy.
 ``loop_input``  before a pass over a range of layers that runs several times: x <- W_in [x ; x0] + step[t], with
                 x0 the embedding output and t the number of the pass (the schedule's stage-call argument).
+``pass_vector`` before a pass over such a range, without a matrix: x <- x + step[t].
 Sums into the residual and the unit norm are fp32.
 """
 from __future__ import annotations
@@ -92,5 +93,27 @@ class LoopInput(StreamStage):
         ops.add_vector(residual, self.step[ctx.call_arg])
 
 
+class PassVector(StreamStage):
+    capturable = True
+
+    def __init__(self, *, width: int, passes: int, step_name: str = "step", dtype: torch.dtype, device: torch.device) -> None:
+        super().__init__(dtype=dtype, device=device)
+        self.width, self.passes, self.step_name = width, passes, step_name
+
+    def weight_specs(self) -> list[WeightSpec]:
+        return [WeightSpec(self.step_name, (self.passes, self.width), std=0.5, role="vector")]
+
+    def bind(self, weights: Mapping[str, torch.Tensor]) -> None:
+        self.step = weights[self.step_name].to(torch.float32).contiguous()
+
+    def forward(self, stream: ResidualStream, ctx: LayerContext) -> None:
+        if not 0 <= ctx.call_arg < self.passes:
+            raise RuntimeError(f"pass {ctx.call_arg} of {self.passes}")
+        # (the last sublayer's pending output and the vector enter the residual in one launch)
+        ops.add_vector(stream.residual, self.step[ctx.call_arg], stream.pending)
+        stream.pending = stream.activation_copy = None
+
+
 register_part("stream_stage", "token_side", TokenSideInput)
 register_part("stream_stage", "loop_input", LoopInput)
+register_part("stream_stage", "pass_vector", PassVector)
