@@ -481,10 +481,17 @@ def _design_configs(DESIGN_WIDTH: int, DESIGN_HEADS: int, kv_heads: int, dense_f
                           {"type": "attention", "mixer": biased, "mlp": grouped},
                           {"type": "latent_attention", "mixer": latent_q, "mlp": grouped},
                           {"type": "attention", "mixer": biased, "mlp": dense}]}
-    return {"zipedra": zipedra, "giforax": giforax, "tibalorn": tibalorn, "vofidra": vofidra, "llama": llama}
+    # Bodopel beside Tibalorn (the closest: grouped attention with biases and an element-wise gate inside a window of the same
+    # size, the same squared-relu feed-forward, short convolutions) and the same Llama: four layers, the middle two as a loop
+    # of one pass (four layer runs, with the pass's vector once)
+    mixed = {"heads": DESIGN_HEADS, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0, "mask": {"size": 512}}
+    bodopel = {"architecture": "Bodopel", "vocab": DESIGN_VOCAB, "width": DESIGN_WIDTH, "max_positions": 8192, "norm": {"eps": 1e-6},
+               "embedding": {"scale": 8.0}, "canon": {"taps": 4}, "loop": {"start": 1, "stop": 3, "times": 1},
+               "layers": [{"type": "attention", "mixer": mixed, "mlp": dense} for _ in range(DESIGN_LAYERS)]}
+    return {"zipedra": zipedra, "giforax": giforax, "tibalorn": tibalorn, "vofidra": vofidra, "bodopel": bodopel, "llama": llama}
 
 
-DESIGN_ALSO_BESIDE = {"vofidra": ("zipedra",)}      # the closest design of the package, measured in the same call
+DESIGN_ALSO_BESIDE = {"vofidra": ("zipedra",), "bodopel": ("tibalorn",)}      # the closest design of the package, measured in the same call
 
 
 def run_design(args) -> dict:
@@ -546,6 +553,10 @@ def run_design(args) -> dict:
                                ["expert-product"]),
                    "tibalorn": (["pooled-window-attention"], ["state-space", "--heads", str(args.design_width // 32)],
                                 ["sigmoid-attention"], ["gated-recurrence"], ["layer-tails"]),
+                   "bodopel": (["talking-heads", "--heads", str(args.design_width // 128), "--kv-heads", str(args.design_width // 256)],
+                               ["pooled-window-attention", "--heads", str(args.design_width // 128), "--kv-heads", str(args.design_width // 256)],
+                               ["input-conv", "--hidden", str(args.design_width)],
+                               ["state-space", "--heads", str(args.design_width // 32)]),
                    "vofidra": (["biased-attention", "--heads", str(args.design_width // 128), "--kv-heads", str(args.design_width // 256)],
                                ["latent-attention", "--heads", str(args.design_width // 128)],
                                ["hyper-streams", "--hidden", str(args.design_width)],
@@ -657,7 +668,7 @@ def main(argv=None) -> int:
     parser.add_argument("--gemm-backend", choices=["auto", "tcgen05", "library"], default="auto")
     parser.add_argument("--workloads", nargs="*", default=list(WORKLOADS), choices=list(WORKLOADS),
                         help="serving workloads of the smaller sizes to add to points")
-    parser.add_argument("--design", choices=["zipedra", "giforax", "tibalorn", "vofidra"], default=None,
+    parser.add_argument("--design", choices=["zipedra", "giforax", "tibalorn", "vofidra", "bodopel"], default=None,
                         help="instead of the headline run: prefill and decode throughput of this design at layer sizes that "
                              "resemble a real model's, beside the closest Llama, and its kernels against the roofline")
     parser.add_argument("--design-width", type=int, default=DESIGN_WIDTH,

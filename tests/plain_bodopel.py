@@ -88,7 +88,8 @@ def attention(h, w, p, m, eps):
     scores = capped(torch.einsum("ihd,jhd->hij", q, kh) * m["scale"], m["softcap"])
     distance = (torch.arange(T)[:, None] - torch.arange(T)[None, :]).clamp(min=0)
     scores = scores - distance_loss(w[p + "r1"], w[p + "r2"], distance)
-    weights = mix_heads(window_weights(scores, m["mask"]["size"]), w[p + "talk"])
+    window = T if m["mask"] is None else m["mask"]["size"]
+    weights = mix_heads(window_weights(scores, window), w[p + "talk"])
     rows = torch.einsum("hij,jhd->ihd", weights, vh).reshape(T, H * dv)
     return (rows * torch.sigmoid(h @ w[p + "g"].T)) @ w[p + "o"].T
 

@@ -161,7 +161,8 @@ def run_trace_program(folder, dtype: str, max_tokens: int, steps, out_dir: Path,
     finally:
         if proc.poll() is None:
             proc.kill()
-    vocab = json.loads((Path(folder) / "config.json").read_text())["vocab_size"]
+    config = json.loads((Path(folder) / "config.json").read_text())
+    vocab = config.get("vocab_size") or config["vocab"]
     out = {}
     for step in steps:
         wanted = sum(len(e["want"]) for e in step["entries"])

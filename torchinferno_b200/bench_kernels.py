@@ -13,6 +13,8 @@
     python -m torchinferno_b200.bench_kernels layer-tails --rows 2048
     python -m torchinferno_b200.bench_kernels pooled-window-attention --tokens 2048 --batch 8 --context 2048 --window 512 --pool 64
     python -m torchinferno_b200.bench_kernels state-space --tokens 2048 --batch 8
+    python -m torchinferno_b200.bench_kernels talking-heads --tokens 2048 --batch 8 --context 2048 --window 512
+    python -m torchinferno_b200.bench_kernels input-conv --rows 2048
 
 Each run prints one JSON line per case: microseconds (median of CUDA-event timings, an L2 flush
 between iterations), the bytes or flops the kernel has to move or do, and the fraction of the
@@ -510,6 +512,86 @@ def run_biased_attention(args) -> None:
     report("qk_norm_append[prompt, weights and temperature]", timer(fn), bytes_moved=n * ((h + k) * d + k * v) * 4, tokens=n)
 
 
+def run_talking_heads(args) -> None:
+    """The windowed attention whose softmax weights are mixed across the heads on a prompt of --tokens (flops: both products
+    and the mix over the keys a query sees) and on --batch single tokens at --context (bytes: the keys and values inside every
+    request's window once); then the launch ahead of it (biases, norms over the whole rows, the store into the pages)."""
+    h, k, d, v, page, window = args.heads, args.kv_heads, args.head_dim, args.value_dim, args.page_size, args.window
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device="cuda")
+    timer = Timer(args.iters)
+
+    def pages(n_entries, entries_per):
+        per = -(-entries_per // page)
+        pool_ = (torch.randn(n_entries * per, k * page * (d + v), device="cuda") * 0.5).to(torch.bfloat16)
+        table = torch.randperm(n_entries * per, device="cuda", dtype=torch.int32).view(n_entries, per).contiguous()
+        return pool_[:, :k * page * d].unflatten(1, (k, page, d)), pool_[:, k * page * d:].unflatten(1, (k, page, v)), table
+
+    talk = (torch.eye(h, device="cuda") + 0.2 * torch.randn(h, h, device="cuda")).to(torch.bfloat16)
+    padded = 16 if h <= 16 else 32 if h <= 32 else 64
+    talk_hi = torch.zeros(padded, padded, dtype=torch.bfloat16, device="cuda")
+    talk_hi[:h, :h] = talk
+    bias = -torch.rand(h, 1, device="cuda") * torch.log1p(torch.rand(h, 1, device="cuda") * torch.arange(window, device="cuda"))
+    for mode in ("prompt", "single tokens"):
+        n_entries, ctx = (1, args.tokens) if mode == "prompt" else (args.batch, args.context)
+        keys, values, table = pages(n_entries, ctx)
+        n = ctx if mode == "prompt" else n_entries
+        q = torch.randn(n, h * d, device="cuda").to(torch.bfloat16)
+        gate = torch.randn(n, h * v, device="cuda").to(torch.bfloat16)
+        out = torch.empty(n, h * v, dtype=torch.bfloat16, device="cuda")
+        seen = min(ctx, window)
+        if mode == "prompt":
+            q_start, kv_start, slots, positions, max_q = i32([0, n]), i32([0]), i32([0]), i32(list(range(n))), n
+            pairs = seen * (seen + 1) / 2 + (ctx - seen) * seen
+            flops, moved = 2 * h * (d + v + h) * pairs, None
+        else:
+            q_start, kv_start, slots, max_q = i32(list(range(n + 1))), i32([ctx - 1] * n), i32(list(range(n))), 1
+            positions = kv_start
+            flops, moved = None, n * seen * k * (d + v) * 2
+        for scratch in ([None] if mode == "single tokens" or not args.scratch_mb else [mb << 20 for mb in args.scratch_mb]):
+            for tiles in ([None] if mode == "prompt" or not args.tiles else args.tiles):
+                fn = lambda: ops.talking_heads_attention(
+                    q, out, q_start, kv_start, slots, positions, keys, values, table, n_entries, max_q, h, k, window=window, scale=0.09,
+                    softcap=args.softcap, bias=bias, talk=talk.float(), talk_hi=talk_hi, gate=gate, max_kv_len=ctx, scratch_bytes=scratch,
+                    tiles_per_part=tiles)
+                report(f"talking_heads_attention[{mode}]", timer(fn), flops=flops, bytes_moved=moved, entries=n_entries, context=ctx,
+                       heads=h, kv_heads=k, head_dim=d, value_dim=v, window=window, **({"scratch_mb": scratch >> 20} if scratch else {}),
+                       **({"tiles_per_part": tiles} if tiles else {}))
+    for n in (args.tokens, args.batch):
+        keys, values, table = pages(1, n)
+        width = (h + k) * d + k * v + h * v
+        proj = torch.randn(n, width, device="cuda").to(torch.bfloat16)
+        q = torch.empty(n, h * d, dtype=torch.bfloat16, device="cuda")
+        positions, token_slot = i32(list(range(n))), i32([0] * n)
+        ones = lambda w: torch.ones(w, device="cuda")
+        params = dict(q_bias=ones(h * d), k_bias=ones(k * d), v_bias=ones(k * v), q_weight=ones(h * d), k_weight=ones(k * d))
+        fn = lambda: ops.row_norm_append(proj, 0, h * d, (h + k) * d, q, keys, values, positions, token_slot, table, h, k, d, v, eps=1e-6, **params)
+        report("row_norm_append", timer(fn), bytes_moved=n * ((h + k) * d + k * v) * 4, tokens=n)
+
+
+def run_input_conv(args) -> None:
+    """The short convolution added to a sublayer's input: on the normed rows of a prompt (bytes: rows read and written), and
+    with the residual sum and the norm on single tokens; beside them the residual sum with the norm alone."""
+    w, taps = args.hidden, args.taps
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device="cuda")
+    timer = Timer(args.iters)
+    weight = torch.randn(taps, w, device="cuda")
+    gain = torch.ones(w, device="cuda")
+    for rows in (args.rows, args.batch):
+        x = torch.randn(rows, w, device="cuda").to(torch.bfloat16)
+        out, residual = torch.empty_like(x), torch.randn(rows, w, device="cuda")
+        single = rows == args.batch
+        entries = rows if single else 1
+        state = torch.zeros(entries, (taps - 1) * w, device="cuda")
+        q_start, slots = i32(list(range(rows + 1)) if single else [0, rows]), i32(list(range(entries)))
+        report("input_conv", timer(lambda: ops.input_conv(x, out, weight, state, 0, q_start, slots, entries, 1 if single else rows)),
+               bytes_moved=rows * w * 4 + entries * (taps - 1) * w * 8, rows=rows, hidden=w, taps=taps)
+        if single:
+            report("norm_conv_step", timer(lambda: ops.norm_conv_step(x, residual, gain, 1e-6, weight, state, 0, slots, out)),
+                   bytes_moved=rows * w * 12 + rows * (taps - 1) * w * 8, rows=rows, hidden=w, taps=taps)
+        report("add_rmsnorm", timer(lambda: ops.add_rmsnorm(x, residual, gain, 1e-6, out)), bytes_moved=rows * w * 12, rows=rows, hidden=w)
+        report("relu_squared", timer(lambda: ops.relu_squared(x, out)), bytes_moved=rows * w * 4, rows=rows, hidden=w)
+
+
 def run_hyper_streams(args) -> None:
     """A residual in --streams streams: the write of a sublayer's output and the read for the next with the tanh norm in one
     launch (bytes: every stream read and written in fp32, the output rows read, the normed rows written), the read alone,
@@ -688,6 +770,28 @@ def main(argv=None) -> int:
     p.add_argument("--page-size", type=int, default=16)
     p.add_argument("--iters", type=int, default=10)
     p.set_defaults(func=run_biased_attention)
+    p = sub.add_parser("talking-heads")
+    p.add_argument("--tokens", type=int, default=2048)
+    p.add_argument("--batch", type=int, default=8)
+    p.add_argument("--context", type=int, default=2048)
+    p.add_argument("--heads", type=int, default=16)
+    p.add_argument("--kv-heads", type=int, default=8)
+    p.add_argument("--head-dim", type=int, default=128)
+    p.add_argument("--value-dim", type=int, default=128)
+    p.add_argument("--window", type=int, default=512)
+    p.add_argument("--softcap", type=float, default=50.0)
+    p.add_argument("--page-size", type=int, default=16)
+    p.add_argument("--scratch-mb", type=int, nargs="*", default=None, help="try these limits of a portion's scratch")
+    p.add_argument("--tiles", type=int, nargs="*", default=None, help="try these numbers of key tiles per block of a single token")
+    p.add_argument("--iters", type=int, default=10)
+    p.set_defaults(func=run_talking_heads)
+    p = sub.add_parser("input-conv")
+    p.add_argument("--rows", type=int, default=2048)
+    p.add_argument("--batch", type=int, default=8)
+    p.add_argument("--hidden", type=int, default=2048)
+    p.add_argument("--taps", type=int, default=4)
+    p.add_argument("--iters", type=int, default=10)
+    p.set_defaults(func=run_input_conv)
     p = sub.add_parser("hyper-streams")
     p.add_argument("--rows", type=int, default=2048)
     p.add_argument("--hidden", type=int, default=2048)

@@ -626,8 +626,9 @@ __global__ void __launch_bounds__(kThMixThreads) th_mix_kernel(ThArgs a) {
   }
 }
 
+// (four blocks an SM: the words of sixteen keys are asked for one piece ahead, and other blocks' warps cover the rest)
 template <int DV>
-__global__ void __launch_bounds__(kThThreads) th_values_kernel(__nv_bfloat16* __restrict__ out, ThArgs a) {
+__global__ void __launch_bounds__(kThThreads, 4) th_values_kernel(__nv_bfloat16* __restrict__ out, ThArgs a) {
   pdl_wait();
   pdl_trigger();
   constexpr int VP = DV + 8;
@@ -677,7 +678,7 @@ __global__ void __launch_bounds__(kThThreads) th_values_kernel(__nv_bfloat16* __
   };
 
   const int g8 = lane >> 2, t4 = lane & 3, row_base = warp * 16;
-  int qpos[2], base_of[2];
+  int base_of[2], left[2];          // the tile edge the row's words are counted from, and the query's own place (-1: no row)
   bool live[2];
   const float* words[2];
 #pragma unroll
@@ -685,51 +686,45 @@ __global__ void __launch_bounds__(kThThreads) th_values_kernel(__nv_bfloat16* __
     const int r = row_base + g8 + 8 * h;
     live[h] = r < nrows;
     const int t = live[h] ? r / gc : 0, g = live[h] ? r - t * gc : 0;
-    qpos[h] = pos0 + t;
-    base_of[h] = th_base(qpos[h], a.window);
+    base_of[h] = th_base(pos0 + t, a.window);
+    left[h] = live[h] ? pos0 + t - base_of[h] : -1;
     words[h] = a.scores + ((size_t)(row0 + t0 + t - a.first_token) * H + (kvh * group + g0 + g)) * a.key_span;
   }
-  // the mixed weights of a tile, as the words lie: [kk][row, row + 8 | keys, keys + 8]; words past the query are zeros
-  auto take = [&](int step, uint2 (&f)[4][4]) {
-    const int base = (s_lo + step) * kThKeys;
+  // the mixed weights of sixteen keys, as the words lie: [row, row + 8 | keys, keys + 8]; words outside what the row sees of
+  // its tiles are zeros
+  auto take = [&](int key, uint2 (&f)[4]) {
 #pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      const bool there = step < steps && live[h] && base >= base_of[h] && base <= qpos[h];
-      const uint2* src = reinterpret_cast<const uint2*>(words[h] + (there ? base - base_of[h] : 0) + 2 * t4);
-      const int left = qpos[h] - base - 2 * t4;                  // keys (and one) from this thread's first on
+    for (int h = 0; h < 2; ++h)
 #pragma unroll
-      for (int kk = 0; kk < 4; ++kk)
-#pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int at = kk * 16 + half * 8;
-          f[kk][h + 2 * half] = there && at <= left ? src[at / 2] : make_uint2(0u, 0u);
-        }
-    }
+      for (int half = 0; half < 2; ++half) {
+        const int at = key + half * 8 + 2 * t4 - base_of[h];
+        f[h + 2 * half] = at >= 0 && at <= left[h] ? *reinterpret_cast<const uint2*>(words[h] + at) : make_uint2(0u, 0u);
+      }
   };
   float o[DV / 8][4];
 #pragma unroll
   for (int n = 0; n < DV / 8; ++n)
 #pragma unroll
     for (int c = 0; c < 4; ++c) o[n][c] = 0.f;
-  uint2 now[4][4], next[4][4];
+  uint2 now[4], next[4];
   fetch(0, 0);
-  take(0, now);
+  take(s_lo * kThKeys, now);
   for (int step = 0; step < steps; ++step) {
     const int stage = step & 1;
     if (step + 1 < steps) fetch(stage ^ 1, step + 1);
     else cp_async_commit();
-    take(step + 1, next);
     cp_async_wait<1>();
     __syncthreads();
     if (row_base < nrows) {
       const __nv_bfloat16* vt = v_s + (size_t)stage * kThKeys * VP;
 #pragma unroll
       for (int kk = 0; kk < 4; ++kk) {
+        take((s_lo + step) * kThKeys + (kk + 1) * 16, next);
         uint32_t p_hi[4], p_lo[4];
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-          p_hi[i] = __byte_perm(now[kk][i].x, now[kk][i].y, 0x5410);
-          p_lo[i] = __byte_perm(now[kk][i].x, now[kk][i].y, 0x7632);
+          p_hi[i] = __byte_perm(now[i].x, now[i].y, 0x5410);
+          p_lo[i] = __byte_perm(now[i].x, now[i].y, 0x7632);
         }
 #pragma unroll
         for (int dn = 0; dn < DV / 16; ++dn) {
@@ -740,13 +735,11 @@ __global__ void __launch_bounds__(kThThreads) th_values_kernel(__nv_bfloat16* __
           mma_bf16(o[2 * dn], p_lo, bv[0], bv[1]);
           mma_bf16(o[2 * dn + 1], p_lo, bv[2], bv[3]);
         }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) now[i] = next[i];
       }
     }
     __syncthreads();      // the stage is free for the fetch after next
-#pragma unroll
-    for (int kk = 0; kk < 4; ++kk)
-#pragma unroll
-      for (int i = 0; i < 4; ++i) now[kk][i] = next[kk][i];
   }
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
