@@ -15,7 +15,7 @@ namespace tib {
 
 constexpr int kIcRegTaps = 8;          // taps held in registers; longer convolutions read their rows again
 constexpr int kIcThreads = 128;
-constexpr int kIcSegment = 16;         // tokens a thread walks
+constexpr int kIcSegment = 16;         // tokens a thread walks (at least the kIcRegTaps - 1 rows that are carried)
 
 struct InputConvArgs {
   const float* weight;                                     // [taps][width]
@@ -170,16 +170,7 @@ norm_conv_step_x8_kernel(const __nv_bfloat16* __restrict__ delta, __nv_bfloat16*
   const int row = blockIdx.x, c = threadIdx.x * 8, carried = a.taps - 1;
   const bool active = c < a.width;
   float4 g0, g1, w[MAXT][2], p[MAXT][2];
-  pdl_wait();
-  pdl_trigger();
-  float* st = a.state + (size_t)a.slots[row] * a.state_stride + a.state_off + c;
-  float h[8];
-  float ss = 0.f;
-  if (active) {
-    float* res = a.residual + (size_t)row * a.width + c;
-    const float4 r0 = *reinterpret_cast<const float4*>(res), r1 = *reinterpret_cast<const float4*>(res + 4);
-    uint4 raw = make_uint4(0, 0, 0, 0);
-    if (delta) raw = *reinterpret_cast<const uint4*>(delta + (size_t)row * a.width + c);
+  if (active) {        // (the weights are on their way while the kernel before this one drains)
     g0 = *reinterpret_cast<const float4*>(a.norm_weight + c);
     g1 = *reinterpret_cast<const float4*>(a.norm_weight + c + 4);
 #pragma unroll
@@ -188,11 +179,24 @@ norm_conv_step_x8_kernel(const __nv_bfloat16* __restrict__ delta, __nv_bfloat16*
         w[k][0] = *reinterpret_cast<const float4*>(a.weight + (size_t)k * a.width + c);
         w[k][1] = *reinterpret_cast<const float4*>(a.weight + (size_t)k * a.width + c + 4);
       }
+    }
+  }
+  pdl_wait();
+  pdl_trigger();
+  float* st = a.state + (size_t)a.slots[row] * a.state_stride + a.state_off + c;
+  float h[8];
+  float ss = 0.f;
+  if (active) {
+#pragma unroll
+    for (int k = 0; k < MAXT; ++k)
       if (k < carried) {
         p[k][0] = *reinterpret_cast<const float4*>(st + (size_t)k * a.width);
         p[k][1] = *reinterpret_cast<const float4*>(st + (size_t)k * a.width + 4);
       }
-    }
+    float* res = a.residual + (size_t)row * a.width + c;
+    const float4 r0 = *reinterpret_cast<const float4*>(res), r1 = *reinterpret_cast<const float4*>(res + 4);
+    uint4 raw = make_uint4(0, 0, 0, 0);
+    if (delta) raw = *reinterpret_cast<const uint4*>(delta + (size_t)row * a.width + c);
     h[0] = r0.x; h[1] = r0.y; h[2] = r0.z; h[3] = r0.w; h[4] = r1.x; h[5] = r1.y; h[6] = r1.z; h[7] = r1.w;
     if (delta) {
       const __nv_bfloat162* d2 = reinterpret_cast<const __nv_bfloat162*>(&raw);

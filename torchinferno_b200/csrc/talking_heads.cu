@@ -98,93 +98,86 @@ template <int VEC> __device__ __forceinline__ void th_load_f32(const float* p, f
 }
 
 constexpr int kThAppendThreads = 256;
-constexpr int kThAppendKeep = 4;      // pieces of a row a thread holds between the two passes (the rest is read again)
+constexpr int kThAppendKeep = 2;      // pieces of a row a thread holds between the two passes (the rest is read again)
 
-// One block per token.  VEC 8: bf16, every width a multiple of 8 (a piece of eight never crosses a head's edge).
+// grid (tokens, 3): a block each for a token's q, k and v.  VEC 8: bf16, every width a multiple of 8 (a piece of eight never
+// crosses a head's edge).
 template <typename T, int VEC>
 __global__ void __launch_bounds__(kThAppendThreads) th_append_kernel(const T* __restrict__ proj, T* __restrict__ q_out, ThAppendArgs a) {
   __shared__ float scratch[33];
-  const int t = blockIdx.x;
+  const int t = blockIdx.x, part = blockIdx.y;         // 0: q, 1: k, 2: v
+  const float* bias = part == 0 ? a.q_bias : part == 1 ? a.k_bias : a.v_bias;
+  const float* weight = part == 0 ? a.q_weight : part == 1 ? a.k_weight : nullptr;
+  const int head_width = part == 2 ? a.vdim : a.dim, width = (part == 0 ? a.heads : a.kv_heads) * head_width;
+  const T* src = proj + (size_t)t * a.ld + (part == 0 ? a.q_off : part == 1 ? a.k_off : a.v_off);
   pdl_wait();
   pdl_trigger();
-  const int pos = a.positions[t];
-  const int* table = a.cache.block_table + (size_t)a.token_slot[t] * a.cache.table_stride;
-  const int page = th_page(a.cache, table, pos, threadIdx.x == 0 ? a.error_word : nullptr, 0x30000 + (t & 0xffff));
-  const int in_page = pos % a.cache.page_size;
-  const T* row = proj + (size_t)t * a.ld;
-  T* k_dst = page < 0 ? nullptr : reinterpret_cast<T*>(a.keys) + (size_t)page * a.cache.page_stride;
-  T* v_dst = page < 0 ? nullptr : reinterpret_cast<T*>(a.values) + (size_t)page * a.cache.page_stride;
-#pragma unroll 1
-  for (int part = 0; part < 2; ++part) {               // q, then k
-    const int width = (part == 0 ? a.heads : a.kv_heads) * a.dim;
-    const T* src = row + (part == 0 ? a.q_off : a.k_off);
-    const float* bias = part == 0 ? a.q_bias : a.k_bias;
-    const float* weight = part == 0 ? a.q_weight : a.k_weight;
-    float kept[kThAppendKeep][VEC];
-    auto biased = [&](int e, float (&v)[VEC]) {
-      th_load<T, VEC>(src + e, v);
-      if (bias) {
-        float b[VEC];
-        th_load_f32<VEC>(bias + e, b);
+  T* dst = q_out + (size_t)t * width;                  // (k and v: the token's row in the first head of its page)
+  if (part > 0) {
+    const int pos = a.positions[t];
+    const int* table = a.cache.block_table + (size_t)a.token_slot[t] * a.cache.table_stride;
+    const int page = th_page(a.cache, table, pos, threadIdx.x == 0 ? a.error_word : nullptr, 0x30000 + (t & 0xffff));
+    if (page < 0) return;                              // (the whole block)
+    dst = reinterpret_cast<T*>(part == 1 ? a.keys : a.values) + (size_t)page * a.cache.page_stride + (size_t)(pos % a.cache.page_size) * head_width;
+  }
+  float kept[kThAppendKeep][VEC], gain[kThAppendKeep][VEC];
+  auto biased = [&](int e, float (&v)[VEC]) {
+    th_load<T, VEC>(src + e, v);
+    if (bias) {
+      float b[VEC];
+      th_load_f32<VEC>(bias + e, b);
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) v[i] += b[i];
-      }
-    };
-    float inv = 1.f;
-    float ss = 0.f;
-#pragma unroll
-    for (int n = 0; n < kThAppendKeep; ++n) {
-      const int e = (n * kThAppendThreads + threadIdx.x) * VEC;
-      if (e < width) {
-        biased(e, kept[n]);
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) ss = fmaf(kept[n][i], kept[n][i], ss);
-      }
+      for (int i = 0; i < VEC; ++i) v[i] += b[i];
     }
-    for (int e = (kThAppendKeep * kThAppendThreads + threadIdx.x) * VEC; e < width; e += kThAppendThreads * VEC) {
+  };
+  auto leave = [&](int e, const float (&v)[VEC]) {
+    if (part == 0) th_store<T, VEC>(dst + e, v);
+    else {
+      const int h = e / head_width;
+      th_store<T, VEC>(dst + (size_t)h * a.cache.page_size * head_width + (e - h * head_width), v);
+    }
+  };
+  float ss = 0.f;
+#pragma unroll
+  for (int n = 0; n < kThAppendKeep; ++n) {
+    const int e = (n * kThAppendThreads + threadIdx.x) * VEC;
+    if (e < width) {
+      biased(e, kept[n]);
+      if (weight) th_load_f32<VEC>(weight + e, gain[n]);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) ss = fmaf(kept[n][i], kept[n][i], ss);
+    }
+  }
+  constexpr int FIRST = kThAppendKeep * kThAppendThreads * VEC;
+  if (weight)
+    for (int e = FIRST + threadIdx.x * VEC; e < width; e += kThAppendThreads * VEC) {
       float v[VEC];
       biased(e, v);
 #pragma unroll
       for (int i = 0; i < VEC; ++i) ss = fmaf(v[i], v[i], ss);
     }
-    if (weight) inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)width + a.eps);
-    auto leave = [&](int e, float (&v)[VEC]) {
+  const float inv = weight ? 1.f / sqrtf(block_sum(ss, scratch) / (float)width + a.eps) : 1.f;
+#pragma unroll
+  for (int n = 0; n < kThAppendKeep; ++n) {
+    const int e = (n * kThAppendThreads + threadIdx.x) * VEC;
+    if (e < width) {
       if (weight) {
-        float g[VEC];
-        th_load_f32<VEC>(weight + e, g);
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) v[i] = v[i] * inv * g[i];
+        for (int i = 0; i < VEC; ++i) kept[n][i] = kept[n][i] * inv * gain[n][i];
       }
-      if (part == 0) th_store<T, VEC>(q_out + (size_t)t * width + e, v);
-      else if (k_dst) {
-        const int h = e / a.dim;
-        th_store<T, VEC>(k_dst + ((size_t)h * a.cache.page_size + in_page) * a.dim + (e - h * a.dim), v);
-      }
-    };
-#pragma unroll
-    for (int n = 0; n < kThAppendKeep; ++n) {
-      const int e = (n * kThAppendThreads + threadIdx.x) * VEC;
-      if (e < width) leave(e, kept[n]);
-    }
-    for (int e = (kThAppendKeep * kThAppendThreads + threadIdx.x) * VEC; e < width; e += kThAppendThreads * VEC) {
-      float v[VEC];
-      biased(e, v);
-      leave(e, v);
+      leave(e, kept[n]);
     }
   }
-  if (v_dst) {
-    for (int e = threadIdx.x * VEC; e < a.kv_heads * a.vdim; e += kThAppendThreads * VEC) {
-      float v[VEC];
-      th_load<T, VEC>(row + a.v_off + e, v);
-      if (a.v_bias) {
-        float b[VEC];
-        th_load_f32<VEC>(a.v_bias + e, b);
+  for (int e = FIRST + threadIdx.x * VEC; e < width; e += kThAppendThreads * VEC) {
+    float v[VEC];
+    biased(e, v);
+    if (weight) {
+      float g[VEC];
+      th_load_f32<VEC>(weight + e, g);
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) v[i] += b[i];
-      }
-      const int h = e / a.vdim;
-      th_store<T, VEC>(v_dst + ((size_t)h * a.cache.page_size + in_page) * a.vdim + (e - h * a.vdim), v);
+      for (int i = 0; i < VEC; ++i) v[i] = v[i] * inv * g[i];
     }
+    leave(e, v);
   }
 }
 
@@ -936,18 +929,44 @@ __global__ void __launch_bounds__(kThThreads) th_step_values_kernel(__nv_bfloat1
   pdl_wait();
   pdl_trigger();
   if (tile_lo >= tile_hi) return;
-  for (int h = tid; h < H; h += kThThreads) {
-    const float* ml = a.part_ml + ((size_t)row0 * a.n_parts * H + h) * 2;
-    float top = -CUDART_INF_F, sum = 0.f;
-    for (int p = 0; p < parts; ++p) top = fmaxf(top, ml[(size_t)p * H * 2]);
-    for (int p = 0; p < parts; ++p) {
-      const float m = ml[(size_t)p * H * 2];
-      sum += m == -CUDART_INF_F ? 0.f : ml[(size_t)p * H * 2 + 1] * exp2f(m - top);
+  const int pair = tid & 63, half = tid >> 6;          // mix: key and half of the heads; values: two columns and half of the keys
+  const float* words = a.scores + (size_t)row0 * H * a.key_span + pair;
+  // the first scores are on their way while the parts' denominators are added up
+  constexpr int AHEAD = 8;
+  float ahead[AHEAD];
+  auto ask = [&](int tile, int i0) {
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i) {
+      const int h = half + 2 * (i0 + i);
+      if (h < H) ahead[i] = words[(size_t)h * a.key_span + tile * kThKeys];
     }
-    lse_s[h] = top + log2f(sum);
+  };
+  ask(tile_lo, 0);
+  // a warp per head, a lane per part (parts beyond 32 in rounds), four heads in flight
+  for (int h0 = (tid >> 5) * 4; h0 < H; h0 += 16) {
+    const int lane = tid & 31;
+    float top[4], sum[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { top[i] = -CUDART_INF_F; sum[i] = 0.f; }
+    for (int p0 = 0; p0 < parts; p0 += 32) {
+      float2 ml[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        ml[i] = p0 + lane < parts && h0 + i < H
+            ? *reinterpret_cast<const float2*>(a.part_ml + (((size_t)row0 * a.n_parts + p0 + lane) * H + h0 + i) * 2)
+            : make_float2(-CUDART_INF_F, 0.f);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float high = fmaxf(top[i], warp_max(ml[i].x)), base = high == -CUDART_INF_F ? 0.f : high;
+        sum[i] = sum[i] * exp2f(top[i] - base) + warp_sum(ml[i].y * exp2f(ml[i].x - base));
+        top[i] = high;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      if (lane == 0 && h0 + i < H) lse_s[h0 + i] = top[i] + log2f(sum[i]);
   }
   __syncthreads();
-  const int pair = tid & 63, half = tid >> 6;          // mix: key and half of the heads; values: two columns and half of the keys
   float o[GC][2];
 #pragma unroll
   for (int g = 0; g < GC; ++g) o[g][0] = o[g][1] = 0.f;
@@ -957,16 +976,20 @@ __global__ void __launch_bounds__(kThThreads) th_step_values_kernel(__nv_bfloat1
       fetch(tile);
     }
     {
-      const float* s = a.scores + (size_t)row0 * H * a.key_span + tile * kThKeys + pair;
       float mixed[GC];
 #pragma unroll
       for (int g = 0; g < GC; ++g) mixed[g] = 0.f;
-#pragma unroll 4
-      for (int h = half; h < H; h += 2) {
-        const float w = exp2f(s[(size_t)h * a.key_span] - lse_s[h]);
+      for (int i0 = 0; half + 2 * i0 < H; i0 += AHEAD) {
+        if (tile > tile_lo || i0 > 0) ask(tile, i0);
 #pragma unroll
-        for (int g = 0; g < GC; ++g)
-          if (g < group) mixed[g] = fmaf(talk_s[g * H + h], w, mixed[g]);
+        for (int i = 0; i < AHEAD; ++i) {
+          const int h = half + 2 * (i0 + i);
+          if (h >= H) continue;
+          const float w = exp2f(ahead[i] - lse_s[h]);
+#pragma unroll
+          for (int g = 0; g < GC; ++g)
+            if (g < group) mixed[g] = fmaf(talk_s[g * H + h], w, mixed[g]);
+        }
       }
 #pragma unroll
       for (int g = 0; g < GC; ++g) mix_s[(half * GC + g) * kThKeys + pair] = mixed[g];
@@ -1133,11 +1156,11 @@ TIB_API int tib_row_norm_append(const void* proj, int64_t ld, int q_off, int k_o
   const bool eights = dim % 8 == 0 && vdim % 8 == 0 && ld % 8 == 0 && q_off % 8 == 0 && k_off % 8 == 0 && v_off % 8 == 0 &&
                       page_stride % 8 == 0 && (bits & 15) == 0;
   if (dtype == TIB_F32)
-    TIB_LAUNCH_DEPENDENT((th_append_kernel<float, 1>), n_tokens, kThAppendThreads, 0, stream, (const float*)proj, (float*)q_out, a);
+    TIB_LAUNCH_DEPENDENT((th_append_kernel<float, 1>), dim3(n_tokens, 3), kThAppendThreads, 0, stream, (const float*)proj, (float*)q_out, a);
   else if (dtype == TIB_BF16 && eights)
-    TIB_LAUNCH_DEPENDENT((th_append_kernel<__nv_bfloat16, 8>), n_tokens, kThAppendThreads, 0, stream, (const __nv_bfloat16*)proj, (__nv_bfloat16*)q_out, a);
+    TIB_LAUNCH_DEPENDENT((th_append_kernel<__nv_bfloat16, 8>), dim3(n_tokens, 3), kThAppendThreads, 0, stream, (const __nv_bfloat16*)proj, (__nv_bfloat16*)q_out, a);
   else if (dtype == TIB_BF16)
-    TIB_LAUNCH_DEPENDENT((th_append_kernel<__nv_bfloat16, 1>), n_tokens, kThAppendThreads, 0, stream, (const __nv_bfloat16*)proj, (__nv_bfloat16*)q_out, a);
+    TIB_LAUNCH_DEPENDENT((th_append_kernel<__nv_bfloat16, 1>), dim3(n_tokens, 3), kThAppendThreads, 0, stream, (const __nv_bfloat16*)proj, (__nv_bfloat16*)q_out, a);
   else
     return TIB_E_DTYPE;
   return TIB_OK;
