@@ -11,12 +11,13 @@ future of a request reserved at admission
 What is different here:
 
 * cache layers are put in **groups** by what they keep (kv_heads, head_dim,
-  window, stride); every group has a pool, an allocator and block tables of its own;
+  window, kept first tokens, stride); every group has a pool, an allocator and block tables of its own;
   a group with a stride s > 1 holds one entry per full run of s tokens (a pooled
   key and value, say) and takes its pages s times slower than the request grows;
 * pages are taken as tokens arrive (:meth:`CacheManager.extend`), and a group
   with a window gives pages back as soon as the window has passed them
-  (:meth:`CacheManager.release_behind_window`), all others when the request ends;
+  (:meth:`CacheManager.release_behind_window`; pages of first tokens that stay
+  in sight, ``CacheSpec.keep_first``, are kept), all others when the request ends;
 * one layer's pages are laid out ``[pages, 2, kv_heads, page_size, head_dim]``
   so that the keys of one head in one page are contiguous (keys and values may
   differ in width: a page then holds all its keys, then all its values);
@@ -306,10 +307,11 @@ class CacheManager:
             # the next query stands at position `length` and reads keys >= length - window + 1
             first_needed_key = request.length - window + 1
             first_needed_page = max(0, first_needed_key) // self.page_size
+            kept_pages = -(-group.spec.keep_first // self.page_size)      # (tokens every later query still sees)
             while request.first_live[gi] < min(first_needed_page, len(request.pages[gi])):
                 logical = request.first_live[gi]
                 page = request.pages[gi][logical]
-                if page >= 0:
+                if page >= 0 and logical >= kept_pages:
                     group.allocator.release(page)
                     request.pages[gi][logical] = -1
                     group.pending[request.slot * self.max_pages_per_request + logical] = -1

@@ -76,6 +76,9 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(flo
 __device__ __forceinline__ float rope_lo(float lo, float hi, float c, float s) { return __fmaf_rn(lo, c, -__fmul_rn(hi, s)); }
 __device__ __forceinline__ float rope_hi(float lo, float hi, float c, float s) { return __fmaf_rn(hi, c, __fmul_rn(lo, s)); }
 
+// x times the normal distribution's cumulative function at x (the exact form of the Gaussian error linear unit)
+__device__ __forceinline__ float gelu_erf(float x) { return 0.5f * x * (1.f + erff(x * 0.70710678118654752f)); }
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -1,6 +1,6 @@
 // Row-wise pieces that blocks other than the pre-norm one are put together from: sums of two sublayer
-// outputs into the 32-bit residual, a unit norm added to the residual, gates (sigmoid, tanh-GELU times a
-// row of a second embedding table), the square of relu, a scale, and the row pairs a layer that re-reads the
+// outputs into the 32-bit residual, a unit norm added to the residual (with a factor, if need be), gates (sigmoid, tanh-GELU
+// times a row of a second embedding table), the square of relu, the erf form of gelu, a scale, and the row pairs a layer that re-reads the
 // embedding output multiplies.  Statistics, gates and sums are fp32; rows leave in the activation type.
 //
 // In every kernel x / y / g may be float or bf16 in memory (a dtype code each) and may be slices of a wider
@@ -38,9 +38,10 @@ __global__ void add_pair_kernel(float* __restrict__ residual, const void* __rest
   }
 }
 
-// residual[t] += y[t] / sqrt(mean(y[t]^2) + eps) * weight
+// residual[t] += scale * (y[t] / sqrt(mean(y[t]^2) + eps) * weight); optionally the new row also leaves in another type.
 __global__ void unit_norm_add_kernel(float* __restrict__ residual, const void* __restrict__ y, int y_dtype, int64_t ldy,
-                                     const float* __restrict__ weight, int width, float eps) {
+                                     const float* __restrict__ weight, int width, float eps, float scale, void* __restrict__ copy,
+                                     int copy_dtype) {
   pdl_wait();
   pdl_trigger();
   __shared__ float scratch[33];
@@ -51,8 +52,58 @@ __global__ void unit_norm_add_kernel(float* __restrict__ residual, const void* _
     ss += v * v;
   }
   const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
-  for (int c = threadIdx.x; c < width; c += blockDim.x)
-    residual[row * width + c] += load_any(y, y_dtype, row * ldy + c) * inv * weight[c];
+  for (int c = threadIdx.x; c < width; c += blockDim.x) {
+    const float v = fmaf(load_any(y, y_dtype, row * ldy + c) * inv * weight[c], scale, residual[row * width + c]);
+    residual[row * width + c] = v;
+    if (copy) store_any(copy, copy_dtype, row * width + c, v);
+  }
+}
+
+// The same for bf16 rows of a multiple of 8 columns, at most 8 * 1024: a thread keeps its eight elements in registers, and the
+// residual row and the weights are on their way while the row's mean square is summed.
+__global__ void __launch_bounds__(1024)
+unit_norm_add_bf16x8_kernel(float* __restrict__ residual, const __nv_bfloat16* __restrict__ y, int64_t ldy,
+                            const float* __restrict__ weight, int width, float eps, float scale, __nv_bfloat16* __restrict__ copy) {
+  __shared__ float scratch[33];
+  const size_t row = blockIdx.x;
+  const int c = threadIdx.x * 8;
+  const bool active = c < width;
+  float w[8], r[8], v[8];
+  float* res = residual + row * width + c;
+  if (active) {      // (the weights do not depend on the kernel before)
+    const float4 w0 = *reinterpret_cast<const float4*>(weight + c), w1 = *reinterpret_cast<const float4*>(weight + c + 4);
+    w[0] = w0.x; w[1] = w0.y; w[2] = w0.z; w[3] = w0.w; w[4] = w1.x; w[5] = w1.y; w[6] = w1.z; w[7] = w1.w;
+  }
+  pdl_wait();
+  pdl_trigger();
+  float ss = 0.f;
+  if (active) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(y + row * ldy + c);
+    const float4 r0 = *reinterpret_cast<const float4*>(res), r1 = *reinterpret_cast<const float4*>(res + 4);
+    r[0] = r0.x; r[1] = r0.y; r[2] = r0.z; r[3] = r0.w; r[4] = r1.x; r[5] = r1.y; r[6] = r1.z; r[7] = r1.w;
+    const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 f = bf16x2_floats(p[i]);
+      v[2 * i] = f.x;
+      v[2 * i + 1] = f.y;
+      ss = fmaf(f.x, f.x, ss);
+      ss = fmaf(f.y, f.y, ss);
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
+  if (!active) return;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) r[i] = fmaf(v[i] * inv * w[i], scale, r[i]);
+  *reinterpret_cast<float4*>(res) = make_float4(r[0], r[1], r[2], r[3]);
+  *reinterpret_cast<float4*>(res + 4) = make_float4(r[4], r[5], r[6], r[7]);
+  if (copy) {
+    uint4 packed;
+    __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) o[i] = __floats2bfloat162_rn(r[2 * i], r[2 * i + 1]);
+    *reinterpret_cast<uint4*>(copy + row * width + c) = packed;
+  }
 }
 
 // out[t] = f(x[t]) * sigmoid(g[t]);  f = identity (weight null) or the RMS norm with `weight`.  Column c reads gate
@@ -103,6 +154,14 @@ __global__ void relu_squared_kernel(const void* __restrict__ x, int x_dtype, voi
     const float v = fmaxf(load_any(x, x_dtype, i), 0.f);
     store_any(out, out_dtype, i, v * v);
   }
+}
+
+// out = gelu(x) in its erf form, element by element
+__global__ void gelu_kernel(const void* __restrict__ x, int x_dtype, void* __restrict__ out, int out_dtype, int64_t n) {
+  pdl_wait();
+  pdl_trigger();
+  for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x)
+    store_any(out, out_dtype, i, gelu_erf(load_any(x, x_dtype, i)));
 }
 
 // x *= s (fp32), element by element
@@ -175,12 +234,21 @@ TIB_API int tib_add_pair(float* residual, const void* a, int a_dtype, int64_t ld
   return TIB_OK;
 }
 
+// copy: the new residual rows [rows, width] in copy_dtype, or null.
 TIB_API int tib_unit_norm_add(float* residual, const void* y, int y_dtype, int64_t ldy, const float* weight, int rows,
-                              int width, float eps, cudaStream_t stream) {
+                              int width, float eps, float scale, void* copy, int copy_dtype, cudaStream_t stream) {
   if (rows == 0 || width == 0) return TIB_OK;
   if (!residual || !y || !weight || rows < 0 || width < 0) return TIB_E_ARG;
-  if (!known(y_dtype)) return TIB_E_DTYPE;
-  TIB_LAUNCH_DEPENDENT(unit_norm_add_kernel, rows, row_threads(width), 0, stream, residual, y, y_dtype, ldy, weight, width, eps);
+  if (!known(y_dtype) || (copy && !known(copy_dtype))) return TIB_E_DTYPE;
+  const uintptr_t bits = (uintptr_t)residual | (uintptr_t)y | (uintptr_t)weight | (uintptr_t)copy;
+  if (y_dtype == TIB_BF16 && (!copy || copy_dtype == TIB_BF16) && width % 8 == 0 && width <= 8192 && ldy % 8 == 0 && (bits & 15) == 0) {
+    const int threads = (width / 8 + 31) / 32 * 32;
+    TIB_LAUNCH_DEPENDENT(unit_norm_add_bf16x8_kernel, rows, threads, 0, stream, residual, (const __nv_bfloat16*)y, ldy, weight,
+                         width, eps, scale, (__nv_bfloat16*)copy);
+    return TIB_OK;
+  }
+  TIB_LAUNCH_DEPENDENT(unit_norm_add_kernel, rows, row_threads(width), 0, stream, residual, y, y_dtype, ldy, weight, width, eps,
+                       scale, copy, copy_dtype);
   return TIB_OK;
 }
 
@@ -212,6 +280,15 @@ TIB_API int tib_relu_squared(const void* x, int x_dtype, void* out, int out_dtyp
   if (!known(x_dtype) || !known(out_dtype)) return TIB_E_DTYPE;
   const int blocks = (int)(ceil_div64(n, 256) < 148 * 8 ? ceil_div64(n, 256) : 148 * 8);
   TIB_LAUNCH_DEPENDENT(relu_squared_kernel, blocks, 256, 0, stream, x, x_dtype, out, out_dtype, n);
+  return TIB_OK;
+}
+
+TIB_API int tib_gelu(const void* x, int x_dtype, void* out, int out_dtype, int64_t n, cudaStream_t stream) {
+  if (n == 0) return TIB_OK;
+  if (!x || !out || n < 0) return TIB_E_ARG;
+  if (!known(x_dtype) || !known(out_dtype)) return TIB_E_DTYPE;
+  const int blocks = (int)(ceil_div64(n, 256) < 148 * 8 ? ceil_div64(n, 256) : 148 * 8);
+  TIB_LAUNCH_DEPENDENT(gelu_kernel, blocks, 256, 0, stream, x, x_dtype, out, out_dtype, n);
   return TIB_OK;
 }
 

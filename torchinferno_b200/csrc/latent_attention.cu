@@ -12,7 +12,8 @@
 //                     are (2i, 2i+1), or (i, i + n_freq), angle = position * inv_freq[i] in fp32, on the first
 //                     2 * n_freq elements.
 //   latent_attention  causal softmax attention of the folded queries [tokens, heads, rank + rot] (fp32) over
-//                     the paged latent rows; out [tokens, heads, rank] (fp32).  Two kernels:
+//                     the paged latent rows; out [tokens, heads, rank] (fp32).  Optionally the softmax's denominator also
+//                     holds exp(sink[head]), a number without key and value.  Two kernels:
 //                     - CUDA cores, fp32 throughout (the 32-bit path, and every shape): one warp owns one
 //                       (token, head) row and walks the keys in blocks of 32 aligned to absolute positions, so a
 //                       row's arithmetic does not depend on how the batch was cut;
@@ -133,6 +134,7 @@ struct LatentAttnArgs {
   int page_size, num_pages;
   int64_t page_stride;
   float scale;
+  const float* sink;          // [heads] or null: exp(sink[h]) is added to the softmax's denominator
   int head_chunk, q_tile;
   int* error_word;
   // a step of single tokens may cut every context into `n_splits` runs of `blocks_per_split` key blocks, one block
@@ -141,6 +143,14 @@ struct LatentAttnArgs {
   float* partial;
   int n_splits, blocks_per_split;
 };
+
+// What a row's sum of weighted values is multiplied by: 1 / (its weights' sum), the number without a key counted in.  m: the
+// maximum the weights were made against; l: their sum.
+__device__ __forceinline__ float latent_inverse(float m, float l, const float* sink, int head) {
+  if (!sink) return 1.f / l;
+  const float s = sink[head], top = fmaxf(m, s), keep = expf(m - top);
+  return keep / fmaf(l, keep, expf(s - top));
+}
 
 template <typename T, int DPL>
 __global__ void __launch_bounds__(kLatWarps * 32)
@@ -249,7 +259,7 @@ latent_attention_kernel(const float* __restrict__ folded, const T* __restrict__ 
       continue;
     }
     float* dst = out + ((size_t)(row0 + t0 + t) * a.heads + h0 + g) * a.rank;
-    const float inv = 1.f / l[i];
+    const float inv = latent_inverse(m[i], l[i], a.sink, h0 + g);
 #pragma unroll
     for (int j = 0; j < DPL; ++j) {
       const int dd = lane + 32 * j;
@@ -259,7 +269,8 @@ latent_attention_kernel(const float* __restrict__ folded, const T* __restrict__ 
 }
 
 // grid (heads, tokens): out = sum_s w_s acc_s / sum_s w_s l_s with w_s = exp(m_s - max m); a run without keys has m = -inf
-__global__ void latent_merge_kernel(const float* __restrict__ partial, float* __restrict__ out, int heads, int n_splits, int rank) {
+__global__ void latent_merge_kernel(const float* __restrict__ partial, float* __restrict__ out, const float* __restrict__ sink, int heads,
+                                    int n_splits, int rank) {
   pdl_wait();
   pdl_trigger();
   __shared__ float weight[64], sums[64];      // (at most 64 runs)
@@ -279,7 +290,7 @@ __global__ void latent_merge_kernel(const float* __restrict__ partial, float* __
       weight[s] = weight[s] == -CUDART_INF_F ? 0.f : expf(weight[s] - mx);
       total = fmaf(weight[s], sums[s], total);
     }
-    inv_total = 1.f / total;
+    inv_total = latent_inverse(mx, total, sink, blockIdx.x);
   }
   __syncthreads();
   for (int c = threadIdx.x; c < rank; c += blockDim.x) {
@@ -530,7 +541,7 @@ latent_attention_mma_kernel(const float* __restrict__ folded, const __nv_bfloat1
         }
       } else {
         float* dst = out + ((size_t)row0 * a.heads + r0 + r) * a.rank;
-        const float inv = 1.f / l_run[mt][h];
+        const float inv = latent_inverse(m_run[mt][h], l_run[mt][h], a.sink, (r0 + r) % a.heads);
 #pragma unroll
         for (int n = 0; n < 2 * R64; ++n) {
           dst[col0 + n * 8 + 2 * t4] = o[mt][n][2 * h] * inv;
@@ -552,7 +563,7 @@ static int launch_latent_mma(const float* folded, const void* pool, float* out, 
   dim3 grid(a.partial ? a.n_splits : ceil_div(max_q_len * a.heads, rb), n_entries, a.partial ? ceil_div(a.heads, rb) : 1);
   TIB_LAUNCH_DEPENDENT(kern, grid, kMmaWarps * 32, smem, stream, folded, (const __nv_bfloat16*)pool, out, a);
   if (a.partial)
-    TIB_LAUNCH_DEPENDENT(latent_merge_kernel, dim3(a.heads, n_entries), 128, 0, stream, (const float*)a.partial, out, a.heads,
+    TIB_LAUNCH_DEPENDENT(latent_merge_kernel, dim3(a.heads, n_entries), 128, 0, stream, (const float*)a.partial, out, a.sink, a.heads,
                          a.n_splits, a.rank);
   return TIB_OK;
 }
@@ -570,7 +581,7 @@ static int launch_latent_attention(const float* folded, const void* pool, float*
   dim3 grid(a.partial ? a.n_splits : ceil_div(max_q_len, a.q_tile), n_entries, ceil_div(a.heads, a.head_chunk));
   TIB_LAUNCH_DEPENDENT(kern, grid, kLatWarps * 32, smem, stream, folded, (const T*)pool, out, a);
   if (a.partial)
-    TIB_LAUNCH_DEPENDENT(latent_merge_kernel, dim3(a.heads, n_entries), 128, 0, stream, (const float*)a.partial, out, a.heads,
+    TIB_LAUNCH_DEPENDENT(latent_merge_kernel, dim3(a.heads, n_entries), 128, 0, stream, (const float*)a.partial, out, a.sink, a.heads,
                          a.n_splits, a.rank);
   return TIB_OK;
 }
@@ -621,11 +632,11 @@ TIB_API int tib_latent_attention_splits(int n_entries, int heads, int max_kv_len
 
 // folded: [tokens, heads, rank + rot] fp32; pool: pages of [page_size][rank + rot] in `dtype`; out: [tokens, heads, rank] fp32.
 // n_splits > 1 (a step of single tokens only, contexts of at most max_kv_len keys): partial [tokens, heads, n_splits, 2 + rank].
-// force_simt: the CUDA-core kernel also where the tensor-core one takes the shape.
+// sink: [heads] fp32 or null.  force_simt: the CUDA-core kernel also where the tensor-core one takes the shape.
 TIB_API int tib_latent_attention(const float* folded, const void* pool, float* out, const int* q_start, const int* kv_start,
                                  const int* slots, const int* block_table, int table_stride, int n_entries, int max_q_len,
                                  int heads, int rank, int rot, int page_size, int64_t page_stride, int num_pages, float scale,
-                                 float* partial, int n_splits, int max_kv_len, int force_simt, int* error_word, int dtype,
+                                 const float* sink, float* partial, int n_splits, int max_kv_len, int force_simt, int* error_word, int dtype,
                                  cudaStream_t stream) {
   if (n_entries == 0 || max_q_len == 0) return TIB_OK;
   if (!folded || !pool || !out || !q_start || !kv_start || !slots || !block_table) return TIB_E_ARG;
@@ -633,7 +644,7 @@ TIB_API int tib_latent_attention(const float* folded, const void* pool, float* o
   LatentAttnArgs a;
   a.q_start = q_start; a.kv_start = kv_start; a.slots = slots; a.block_table = block_table; a.table_stride = table_stride;
   a.heads = heads; a.rank = rank; a.width = rank + rot; a.page_size = page_size; a.num_pages = num_pages;
-  a.page_stride = page_stride; a.scale = scale; a.error_word = error_word;
+  a.page_stride = page_stride; a.scale = scale; a.sink = sink; a.error_word = error_word;
   a.partial = nullptr; a.n_splits = 1; a.blocks_per_split = 0;
   if (n_splits > 1) {
     if (!partial || max_q_len != 1 || max_kv_len < 1) return TIB_E_ARG;

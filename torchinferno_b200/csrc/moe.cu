@@ -10,7 +10,7 @@
 //                place[pair] = sorted index.  The order inside an expert may differ from run to run; every row
 //                of a product is computed by itself, so no value depends on it
 //   moe_expert_product   y[s] = act(x[src(s)] . W_e^T) for the sorted rows s of expert e; W: [experts, n, k];
-//                act: none, relu^2, silu, or a clamped gated unit over (gate, up) row pairs of W (row 2i = gate i,
+//                act: none, relu^2, silu, gelu (the erf form), or a clamped gated unit over (gate, up) row pairs of W (row 2i = gate i,
 //                row 2i + 1 = up i): g = min(g, limit), u = clamp(u, -limit, limit), y_i = g * sigmoid(alpha * g) * (u + 1),
 //                or the plain gated unit y_i = silu(g) * u over the same pairs; either leaves n / 2 columns.  `row_scale` (per pair, may be null) multiplies the fp32 sums before the
 //                activation: a router weight that belongs on the expert's input.  bf16 operands whose rows are 16-byte aligned run on the tensor cores
@@ -23,7 +23,7 @@
 namespace tib {
 
 // ----------------------------------------------------------- router logits
-// out[t, e] = x[t] . w[e] in fp32 for a handful of rows w (the router, perhaps a gate row behind it): one warp per
+// out[t, e] = x[t] . w[e] (+ bias[e]) in fp32 for a handful of rows w (the router, perhaps a gate row behind it): one warp per
 // row and group of tokens, lanes stride over k (eight at a time where rows are 16-byte aligned), then a butterfly sum per
 // token: the order of every sum is fixed by k and the alignment alone, so a token's logits do not depend on what else is
 // in the step.  (The general fp32 product gives a product
@@ -45,8 +45,8 @@ __device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&v)[8]) {
 
 template <typename TX, bool VEC>
 __global__ void __launch_bounds__(256)
-router_logits_kernel(const TX* __restrict__ x, int64_t ldx, const float* __restrict__ w, float* __restrict__ out, int64_t ldo,
-                     int tokens, int rows, int K) {
+router_logits_kernel(const TX* __restrict__ x, int64_t ldx, const float* __restrict__ w, const float* __restrict__ bias,
+                     float* __restrict__ out, int64_t ldo, int tokens, int rows, int K) {
   pdl_wait();
   pdl_trigger();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
@@ -81,7 +81,7 @@ router_logits_kernel(const TX* __restrict__ x, int64_t ldx, const float* __restr
 #pragma unroll
     for (int i = 0; i < kRouterTokens; ++i) {
       const float v = warp_sum(acc[i]);
-      if (lane == 0 && i < nt) out[(size_t)(t0 + i) * ldo + e] = v;
+      if (lane == 0 && i < nt) out[(size_t)(t0 + i) * ldo + e] = bias ? v + bias[e] : v;
     }
   }
 }
@@ -211,7 +211,8 @@ moe_group_kernel(const int* __restrict__ ids, int pairs, int experts, int* __res
 
 // ---------------------------------------------------------------- products
 constexpr int GM = 64, GN = 64, GK = 16;
-enum MoeAct : int { MOE_ACT_NONE = 0, MOE_ACT_RELU2 = 1, MOE_ACT_SILU = 2, MOE_ACT_GLU_CLAMP = 3, MOE_ACT_SWIGLU = 4 };
+enum MoeAct : int { MOE_ACT_NONE = 0, MOE_ACT_RELU2 = 1, MOE_ACT_SILU = 2, MOE_ACT_GLU_CLAMP = 3, MOE_ACT_SWIGLU = 4, MOE_ACT_GELU = 5 };
+__host__ __device__ constexpr bool moe_act_gated(int act) { return act == MOE_ACT_GLU_CLAMP || act == MOE_ACT_SWIGLU; }
 
 struct MoeEpilogue {
   int act;
@@ -222,6 +223,7 @@ struct MoeEpilogue {
 __device__ __forceinline__ float moe_act(float v, int act) {
   if (act == MOE_ACT_RELU2) { v = fmaxf(v, 0.f); return v * v; }
   if (act == MOE_ACT_SILU) return v / (1.f + expf(-v));
+  if (act == MOE_ACT_GELU) return gelu_erf(v);
   return v;
 }
 // the gated units over (gate, up) row pairs: clamped (see above), or silu(g) * u
@@ -299,7 +301,7 @@ moe_expert_product_kernel(const TX* __restrict__ x, int64_t ldx, const TW* __res
     const int r = ty * 4 + i;
     if (r >= rows) continue;
     const float rs = ep.row_scale ? ep.row_scale[order[first + r]] : 1.f;
-    if (ep.act >= MOE_ACT_GLU_CLAMP) {
+    if (moe_act_gated(ep.act)) {
 #pragma unroll
       for (int j = 0; j < 4; j += 2) {
         const int gn = n0 + tx * 4 + j;
@@ -410,7 +412,7 @@ moe_expert_product_mma_kernel(const __nv_bfloat16* __restrict__ x, int64_t ldx, 
         const int gn = n0 + wn + j * 8 + 2 * t + (c & 1);
         if (r >= rows || gn >= N) continue;
         const float rs = ep.row_scale ? ep.row_scale[order[first + r]] : 1.f;
-        if (ep.act >= MOE_ACT_GLU_CLAMP) {      // (columns 2t and 2t + 1 of a tile sit in one thread: c and c + 1)
+        if (moe_act_gated(ep.act)) {      // (columns 2t and 2t + 1 of a tile sit in one thread: c and c + 1)
           if ((c & 1) == 0 && gn + 1 < N)
             y[(size_t)(first + r) * ldy + (gn >> 1)] = from_f32<TO>(moe_gated(acc[i][j][c] * rs, acc[i][j][c + 1] * rs, ep.act, ep.limit, ep.alpha));
           continue;
@@ -445,8 +447,9 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
 
 using namespace tib;
 
-// x: [tokens, K] (row stride ldx) float or bf16; w: [rows, K] fp32; out: [tokens, rows] fp32 (row stride ldo)
-TIB_API int tib_router_logits(const void* x, int x_dtype, int64_t ldx, const float* w, float* out, int64_t ldo, int tokens,
+// x: [tokens, K] (row stride ldx) float or bf16; w: [rows, K] fp32; bias: [rows] fp32 or null; out: [tokens, rows] fp32 (row
+// stride ldo)
+TIB_API int tib_router_logits(const void* x, int x_dtype, int64_t ldx, const float* w, const float* bias, float* out, int64_t ldo, int tokens,
                               int rows, int K, cudaStream_t stream) {
   if (tokens == 0 || rows == 0) return TIB_OK;
   if (!x || !w || !out || tokens < 0 || rows < 0 || K < 1) return TIB_E_ARG;
@@ -458,7 +461,7 @@ TIB_API int tib_router_logits(const void* x, int x_dtype, int64_t ldx, const flo
   const int64_t xbytes = x_dtype == TIB_F32 ? 4 : 2;
   const bool vec = K % 4 == 0 && (ldx * xbytes) % 16 == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0;
 #define TIB_ROUTER_GO(TX, VEC) \
-  TIB_LAUNCH_DEPENDENT((router_logits_kernel<TX, VEC>), grid, 256, 0, stream, (const TX*)x, ldx, w, out, ldo, tokens, rows, K)
+  TIB_LAUNCH_DEPENDENT((router_logits_kernel<TX, VEC>), grid, 256, 0, stream, (const TX*)x, ldx, w, bias, out, ldo, tokens, rows, K)
   if (x_dtype == TIB_F32) { if (vec) TIB_ROUTER_GO(float, true); else TIB_ROUTER_GO(float, false); }
   else if (x_dtype == TIB_BF16) { if (vec) TIB_ROUTER_GO(__nv_bfloat16, true); else TIB_ROUTER_GO(__nv_bfloat16, false); }
 #undef TIB_ROUTER_GO
@@ -497,7 +500,7 @@ TIB_API int tib_moe_expert_product(const void* x, int x_dtype, int64_t ldx, cons
                                    cudaStream_t stream) {
   if (pairs == 0 || N == 0) return TIB_OK;
   if (!x || !w || !y || !offsets || !order || pairs < 0 || N < 0 || K < 1 || top < 1) return TIB_E_ARG;
-  if (act < MOE_ACT_NONE || act > MOE_ACT_SWIGLU || (act >= MOE_ACT_GLU_CLAMP && N % 2)) return TIB_E_SIZE;
+  if (act < MOE_ACT_NONE || act > MOE_ACT_GELU || (moe_act_gated(act) && N % 2)) return TIB_E_SIZE;
   MoeEpilogue ep;
   ep.act = act; ep.limit = limit; ep.alpha = alpha; ep.row_scale = row_scale;
   const int row_tiles = ceil_div(pairs, GM) + experts;      // at most this many tiles hold a row

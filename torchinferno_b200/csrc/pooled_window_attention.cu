@@ -12,7 +12,8 @@
 //                      exp(sink[h]) added to its denominator; the head's sum of values is turned back by -i over the
 //                      value pairs and multiplied element by element by sigmoid(gate).  Optionally a learned number per
 //                      head and distance, rel_bias[h][min(i - j, span - 1)], is added to a token's score (a design
-//                      without window or blocks passes a window beyond every position and pool 0)
+//                      without window or blocks passes a window beyond every position and pool 0).  Optionally the first
+//                      `keep` tokens of a sequence stay visible to every later query (pool 0)
 //
 // Scores, the softmax, the sums over values, the turning back and the gate are fp32.  Two kernels.  On the CUDA cores
 // (32-bit, any head size) one warp owns one (query token, query head) row from start to end and walks
@@ -196,6 +197,7 @@ struct PwaArgs {
   const int* q_start; const int* kv_start; const int* slots;
   int heads, kv_heads, dim, vdim;
   int window, pool;                  // pool 0: no blocks, only the window
+  int keep;                          // tokens 0 .. keep - 1 are seen from behind the window too (pool 0 only)
   float scale;
   const float* temp; const float* sink;                    // [heads] or null
   const float* vfreq;                                      // [vdim / 2] or null (values were not turned)
@@ -264,10 +266,12 @@ pwa_attention_kernel(const T* __restrict__ q, T* __restrict__ out, PwaArgs a) {
   const int first_key = max(0, pos0 - a.window + 1);
   const int steps_b = (n_blocks + kPwaKeys - 1) / kPwaKeys;
   const int s_lo = first_key / kPwaKeys, s_hi = last_pos / kPwaKeys;
+  const int steps_k = min(s_lo, (a.keep + kPwaKeys - 1) / kPwaKeys);      // kept tokens ahead of the window's first step (pool 0)
 
-  for (int step = 0; step < steps_b + (s_hi - s_lo + 1); ++step) {
+  for (int step = 0; step < steps_b + steps_k + (s_hi - s_lo + 1); ++step) {
     const bool pooled = step < steps_b;
-    const int base = pooled ? step * kPwaKeys : (s_lo + step - steps_b) * kPwaKeys;      // first block / position of the step
+    // first block / position of the step
+    const int base = pooled || step < steps_k ? step * kPwaKeys : (s_lo + step - steps_b - steps_k) * kPwaKeys;
     const PwaCache& c = pooled ? a.blocks : a.tokens;
     const int* table = pooled ? btable : ttable;
     __syncthreads();      // the tiles of the step before are no longer read (and q_s is written)
@@ -275,7 +279,7 @@ pwa_attention_kernel(const T* __restrict__ q, T* __restrict__ out, PwaArgs a) {
     for (int e = threadIdx.x; e < kPwaKeys * (d + dv); e += blockDim.x) {
       const int j = e / (d + dv), dd = e - j * (d + dv);
       const int idx = base + j;
-      const bool wanted = pooled ? idx < n_blocks : (idx <= last_pos && idx >= first_key);
+      const bool wanted = pooled ? idx < n_blocks : (idx <= last_pos && (idx >= first_key || idx < a.keep));
       float val = 0.f;
       if (wanted) {
         const int page = pwa_page(c, table, idx, a.error_word, 0x10000 + entry);
@@ -302,8 +306,8 @@ pwa_attention_kernel(const T* __restrict__ q, T* __restrict__ out, PwaArgs a) {
         allowed = idx < seen;
       } else {
         const int lo = max(0, qpos - a.window + 1);
-        if (base > qpos || base + kPwaKeys - 1 < lo) continue;
-        allowed = idx <= qpos && idx >= lo;
+        if (base > qpos || (base + kPwaKeys - 1 < lo && base >= a.keep)) continue;
+        allowed = idx <= qpos && (idx >= lo || idx < a.keep);
       }
       float s = 0.f;
       const float* qr = q_s + r * d;
@@ -417,13 +421,17 @@ constexpr int kPmRows = 64, kPmKeys = 64, kPmThreads = 128;
 constexpr int kPmFewRowStages = 2;
 constexpr float kLog2e = 1.4426950408889634f;
 
-// REL: the kernel knows the table of biases by distance and contexts shared out over blocks (without it, it is the kernel
-// as the designs without either have always run it, register for register).
-template <int DK, int DV, int ST, bool WT, bool REL>
+// FORM: what the kernel knows beside the window and the blocks (in the plain form it is the kernel as the designs without
+// any of it have always run it, register for register): kPwaRel a table of biases by distance, kPwaKeep first tokens that
+// stay in sight; both know contexts that are shared out over blocks.
+enum { kPwaPlain = 0, kPwaRel = 1, kPwaKeep = 2 };
+
+template <int DK, int DV, int ST, bool WT, int FORM>
 __global__ void __launch_bounds__(kPmThreads)
 pwa_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ out, PwaArgs a) {
   pdl_wait();
   pdl_trigger();
+  constexpr bool REL = FORM == kPwaRel, KEEP = FORM == kPwaKeep, SHARES = FORM != kPwaPlain;
   constexpr int KP = DK + 8, VP = DV + 8;        // padded rows: ldmatrix rows fall in different banks
   extern __shared__ __align__(16) unsigned char sm_raw[];
   __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(sm_raw);          // [64][KP]
@@ -442,7 +450,7 @@ pwa_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __r
   const int row0 = a.q_start[entry];
   const int q_len = a.q_start[entry + 1] - row0;
   // (with the contexts shared out, blockIdx.x counts the parts of a context, and the block's rows are the entry's only ones)
-  const bool shared_out = REL && WT && a.n_splits > 1;
+  const bool shared_out = SHARES && WT && a.n_splits > 1;
   const int t0 = shared_out ? 0 : blockIdx.x * a.q_tile;
   if (t0 >= q_len) return;
   const int nt = min(a.q_tile, q_len - t0);
@@ -459,7 +467,14 @@ pwa_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __r
   const int first_key = max(0, pos0 - a.window + 1);
   const int steps_b = (n_blocks + kPmKeys - 1) / kPmKeys;
   const int s_lo = first_key / kPmKeys, s_hi = last_pos / kPmKeys;
-  const int steps = steps_b + (s_hi - s_lo + 1);
+  const int keep = KEEP ? a.keep : 0;
+  const int steps_k = KEEP ? min(s_lo, (keep + kPmKeys - 1) / kPmKeys) : 0;      // kept tokens' tiles ahead of the window's first
+  const int steps = steps_b + steps_k + (s_hi - s_lo + 1);
+  // first block / position of a step's tile
+  auto tile_base = [&](int step) {
+    if (KEEP) return (step < steps_k ? step : s_lo + step - steps_k) * kPmKeys;      // (no blocks in this form)
+    return (step < steps_b ? step : s_lo + step - steps_b) * kPmKeys;
+  };
   int step_lo = 0, step_hi = steps;                   // this block's share of the tiles
   if (shared_out) {
     const int per = (steps + a.n_splits - 1) / a.n_splits;
@@ -471,10 +486,10 @@ pwa_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __r
   auto locate = [&](int stage, int step, int j) {
     const bool pooled = step < steps_b;
     const PwaCache& c = pooled ? a.blocks : a.tokens;
-    const int idx = (pooled ? step : s_lo + step - steps_b) * kPmKeys + j;
+    const int idx = tile_base(step) + j;
     long long base = -1;
     int row = 0;
-    if (pooled ? idx < n_blocks : (idx <= last_pos && idx >= first_key)) {
+    if (pooled ? idx < n_blocks : (idx <= last_pos && (idx >= first_key || (KEEP && idx < keep)))) {
       const int page = pwa_page(c, pooled ? btable : ttable, idx, a.error_word, 0x10000 + entry);
       if (page >= 0) {
         base = (long long)page * c.page_stride;
@@ -567,9 +582,10 @@ pwa_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __r
 
   auto tile = [&](int stage, int step) {
     const bool pooled = step < steps_b;
-    const int base = (pooled ? step : s_lo + step - steps_b) * kPmKeys;
+    const int base = tile_base(step);
     // (a warp whose rows see nothing of this tile still passes the barriers)
-    const bool any = row_base < nrows && (pooled ? base < warp_seen : (base <= warp_last && base + kPmKeys - 1 >= warp_lo));
+    const bool any = row_base < nrows && (pooled ? base < warp_seen
+                                                : (base <= warp_last && (base + kPmKeys - 1 >= warp_lo || (KEEP && base < keep))));
     if (any) {
       const __nv_bfloat16* kt = k_s + (size_t)stage * kPmKeys * KP;
       const __nv_bfloat16* vt = v_s + (size_t)stage * kPmKeys * VP;
@@ -597,7 +613,7 @@ pwa_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __r
         for (int c = 0; c < 4; ++c) {
           const int h = c >> 1;
           const int idx = base + n * 8 + 2 * t4 + (c & 1);
-          const bool allowed = live[h] && (pooled ? idx < seen[h] : (idx <= qpos[h] && idx >= lo[h]));
+          const bool allowed = live[h] && (pooled ? idx < seen[h] : (idx <= qpos[h] && (idx >= lo[h] || (KEEP && idx < keep))));
           s[n][c] = allowed ? s[n][c] * factor[h] : -CUDART_INF_F;
         }
       if (REL && a.rel_bias && !pooled) {
@@ -845,7 +861,7 @@ pwa_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __r
 }
 
 // Adds the parts of a context that was shared out over blocks, in the order of the parts: out = sum_s o_s 2^(m_s - top)
-// / (sum_s l_s 2^(m_s - top) + 2^(sink - top)).  One block per token, a warp per head.
+// / (sum_s l_s 2^(m_s - top) + 2^(sink - top)), times the gate.  One block per token, a warp per head.
 template <int DV>
 __global__ void __launch_bounds__(128) pwa_merge_kernel(__nv_bfloat16* __restrict__ out, PwaArgs a) {
   pdl_wait();
@@ -875,15 +891,24 @@ __global__ void __launch_bounds__(128) pwa_merge_kernel(__nv_bfloat16* __restric
     const float inv = denom > 0.f ? scale / denom : 0.f;
 #pragma unroll
     for (int j = 0; j < DV / 32; ++j)
-      if (lane + 32 * j < a.vdim) out[(size_t)token * a.heads * a.vdim + (size_t)head * a.vdim + lane + 32 * j] = __float2bfloat16_rn(acc[j] * inv);
+      if (lane + 32 * j < a.vdim) {
+        float v = acc[j] * inv;
+        if (a.gate) {
+          const size_t at = (size_t)token * a.ld_gate + head * a.vdim + lane + 32 * j;
+          const float g = a.gate_dtype == TIB_F32 ? reinterpret_cast<const float*>(a.gate)[at]
+                                                  : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.gate)[at]);
+          v *= 1.f / (1.f + expf(-g));
+        }
+        out[(size_t)token * a.heads * a.vdim + (size_t)head * a.vdim + lane + 32 * j] = __float2bfloat16_rn(v);
+      }
   }
 }
 
-template <int DK, int DV, int ST, bool WT, bool REL>
+template <int DK, int DV, int ST, bool WT, int FORM>
 static int pwa_launch_mma_staged(const void* q, void* out, const PwaArgs& a, dim3 grid, cudaStream_t stream) {
   static_assert(kPmRows * DV * sizeof(float) <= ST * kPmKeys * (DK + 8 + DV + 8) * sizeof(__nv_bfloat16), "the rows' sums fit the stages");
   const size_t smem = sizeof(__nv_bfloat16) * ((size_t)kPmRows * (DK + 8) + ST * (size_t)kPmKeys * (DK + 8) + ST * (size_t)kPmKeys * (DV + 8));
-  auto kern = pwa_attention_mma_kernel<DK, DV, ST, WT, REL>;
+  auto kern = pwa_attention_mma_kernel<DK, DV, ST, WT, FORM>;
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
@@ -907,20 +932,23 @@ static int pwa_launch_mma(const void* q, void* out, PwaArgs a, int n_entries, in
   if ((int64_t)max_q_len * a.group_chunk <= 16) {
     if (a.n_splits > 1) {
       // single tokens whose contexts are shared out over n_splits blocks each; a second kernel adds the parts
-      if (max_q_len != 1 || !a.partial || a.vfreq || a.gate) return TIB_E_ARG;
+      if (max_q_len != 1 || !a.partial || a.vfreq) return TIB_E_ARG;
       grid.x = a.n_splits;
-      const int status = pwa_launch_mma_staged<DK, DV, kPmFewRowStages, true, true>(q, out, a, grid, stream);
+      const int status = a.keep > 0 ? pwa_launch_mma_staged<DK, DV, kPmFewRowStages, true, kPwaKeep>(q, out, a, grid, stream)
+                                    : pwa_launch_mma_staged<DK, DV, kPmFewRowStages, true, kPwaRel>(q, out, a, grid, stream);
       if (status != TIB_OK) return status;
       TIB_LAUNCH_DEPENDENT(pwa_merge_kernel<DV>, a.n_tokens, 128, 0, stream, (__nv_bfloat16*)out, a);
       return TIB_OK;
     }
     a.n_splits = 1;
-    if (a.rel_bias) return pwa_launch_mma_staged<DK, DV, kPmFewRowStages, true, true>(q, out, a, grid, stream);
-    return pwa_launch_mma_staged<DK, DV, 4, true, false>(q, out, a, grid, stream);
+    if (a.keep > 0) return pwa_launch_mma_staged<DK, DV, kPmFewRowStages, true, kPwaKeep>(q, out, a, grid, stream);
+    if (a.rel_bias) return pwa_launch_mma_staged<DK, DV, kPmFewRowStages, true, kPwaRel>(q, out, a, grid, stream);
+    return pwa_launch_mma_staged<DK, DV, 4, true, kPwaPlain>(q, out, a, grid, stream);
   }
   a.n_splits = 1;
-  if (a.rel_bias) return pwa_launch_mma_staged<DK, DV, 2, false, true>(q, out, a, grid, stream);
-  return pwa_launch_mma_staged<DK, DV, 2, false, false>(q, out, a, grid, stream);
+  if (a.keep > 0) return pwa_launch_mma_staged<DK, DV, 2, false, kPwaKeep>(q, out, a, grid, stream);
+  if (a.rel_bias) return pwa_launch_mma_staged<DK, DV, 2, false, kPwaRel>(q, out, a, grid, stream);
+  return pwa_launch_mma_staged<DK, DV, 2, false, kPwaPlain>(q, out, a, grid, stream);
 }
 
 // How many blocks a step of `n_entries` single tokens should share each context of up to `max_kv_len` visible keys out
@@ -1016,15 +1044,16 @@ TIB_API int tib_pool_blocks(const void* k_pages, const void* v_pages, const int*
 // own dtype) or null; temp, sink: [heads] fp32 or null; vfreq: [vdim / 2] fp32 or null.  pool 0: the window alone.
 // rel_bias: [heads, rel_span] fp32 or null: rel_bias[h, min(i - j, rel_span - 1)] is added to the score of token j (not
 // multiplied by scale or temp; blocks get none).  n_splits > 1 (a step of single tokens only, bf16 on the tensor cores, no
-// turned values and no gate): every context is shared out over n_splits blocks, whose sums go through `partial`
+// turned values): every context is shared out over n_splits blocks, whose sums go through `partial`
 // [n_splits, n_tokens, heads, part floats] to a second kernel; n_tokens: rows of q.
+// keep > 0: the first `keep` tokens are seen from behind the window too (no blocks and no rel_bias then).
 // force_simt: the CUDA-core kernel also where the tensor-core kernel would take the step.
 TIB_API int tib_pooled_window_attention(const void* q, void* out, const int* q_start, const int* kv_start, const int* slots,
                                         const void* k_pages, const void* v_pages, const int* block_table, int table_stride,
                                         int page_size, int64_t page_stride, int num_pages, const void* bk_pages,
                                         const void* bv_pages, const int* b_table, int b_table_stride, int b_page_size,
                                         int64_t b_page_stride, int b_num_pages, int n_entries, int max_q_len, int heads,
-                                        int kv_heads, int dim, int vdim, int window, int pool, float scale, const float* temp,
+                                        int kv_heads, int dim, int vdim, int window, int keep, int pool, float scale, const float* temp,
                                         const float* sink, const float* vfreq, const void* gate, int gate_dtype, int64_t ld_gate,
                                         const float* rel_bias, int rel_span, float* partial, int n_splits, int n_tokens,
                                         int* error_word, int dtype, int force_simt, cudaStream_t stream) {
@@ -1035,9 +1064,10 @@ TIB_API int tib_pooled_window_attention(const void* q, void* out, const int* q_s
   if (dim > 256 || vdim > 256 || (vfreq && vdim % 2) || n_entries > 65535) return TIB_E_SIZE;
   if (gate && gate_dtype != TIB_F32 && gate_dtype != TIB_BF16) return TIB_E_DTYPE;
   if (rel_bias && rel_span < 1) return TIB_E_SIZE;
+  if (keep < 0 || (keep > 0 && (pool > 0 || rel_bias))) return TIB_E_SIZE;
   PwaArgs a;
   a.q_start = q_start; a.kv_start = kv_start; a.slots = slots; a.heads = heads; a.kv_heads = kv_heads; a.dim = dim; a.vdim = vdim;
-  a.window = window; a.pool = pool; a.scale = scale; a.temp = temp; a.sink = sink; a.vfreq = vfreq; a.gate = gate;
+  a.window = window; a.keep = keep; a.pool = pool; a.scale = scale; a.temp = temp; a.sink = sink; a.vfreq = vfreq; a.gate = gate;
   a.gate_dtype = gate_dtype; a.ld_gate = ld_gate; a.rel_bias = rel_bias; a.rel_span = rel_span;
   a.tokens = pwa_cache(const_cast<void*>(k_pages), const_cast<void*>(v_pages), block_table, table_stride, page_size, page_stride, num_pages);
   a.blocks = pwa_cache(const_cast<void*>(bk_pages), const_cast<void*>(bv_pages), b_table, b_table_stride, b_page_size, b_page_stride, b_num_pages);

@@ -5,7 +5,8 @@
 //   ssd_scan          per head h (its group g = h / (heads / groups)), S [N, P] in 32-bit, carried per request:
 //                       dt_t = softplus(raw_t + dt_bias[h]);   a_t = exp(-exp(A_log[h]) * dt_t)
 //                       S_t  = a_t * S_(t-1) + dt_t * B_t x_t^T;   y_t = S_t^T C_t + D[h] * x_t
-//   gated_group_norm  out = (y * silu(z)) / rms over each of `parts` equal runs of the row * weight
+//   gated_group_norm  out = (y * silu(z)) / rms over each of `parts` equal runs of the row * weight, or, with the gate behind
+//                     the norm, y / rms over each run * weight * sigmoid(z)
 //
 // Step sizes, decays, the state, the sums over it, the gate and the norm are fp32 in both modes; the convolution
 // accumulates in fp32 and leaves its rows in the activation type.  Every kernel takes the step's ragged batch
@@ -393,7 +394,9 @@ __global__ void __launch_bounds__(256) ssd_fold_runs_kernel(ScanArgs a) {
 }
 
 // -------------------------------------------------------------------------------------------- gate, then norm
-// grid (rows, parts): out[t, c] = v / sqrt(mean over the part of v^2 + eps) * weight[c],  v = y[t, c] * silu(z[t, c])
+// grid (rows, parts): out[t, c] = v / sqrt(mean over the part of v^2 + eps) * weight[c],  v = y[t, c] * silu(z[t, c]);
+// GATE_LAST: v = y[t, c], and the result is multiplied by sigmoid(z[t, c])
+template <bool GATE_LAST>
 __global__ void __launch_bounds__(256)
 gated_group_norm_kernel(const float* __restrict__ y, const void* __restrict__ z, int z_dtype, int64_t ldz, int z_col,
                         const float* __restrict__ weight, float eps, void* __restrict__ out, int out_dtype, int width, int part) {
@@ -404,13 +407,15 @@ gated_group_norm_kernel(const float* __restrict__ y, const void* __restrict__ z,
   const int c0 = blockIdx.y * part;
   float ss = 0.f;
   for (int c = threadIdx.x; c < part; c += blockDim.x) {
-    const float v = y[row * width + c0 + c] * ss_silu(ss_load(z, z_dtype, row * ldz + z_col + c0 + c));
+    const float g = GATE_LAST ? 1.f : ss_silu(ss_load(z, z_dtype, row * ldz + z_col + c0 + c));
+    const float v = y[row * width + c0 + c] * g;
     ss = fmaf(v, v, ss);
   }
   const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)part + eps);
   for (int c = threadIdx.x; c < part; c += blockDim.x) {
-    const float v = y[row * width + c0 + c] * ss_silu(ss_load(z, z_dtype, row * ldz + z_col + c0 + c));
-    ss_store(out, out_dtype, row * width + c0 + c, v * inv * weight[c0 + c]);
+    const float zc = ss_load(z, z_dtype, row * ldz + z_col + c0 + c), yc = y[row * width + c0 + c];
+    const float v = GATE_LAST ? yc * inv * weight[c0 + c] / (1.f + expf(-zc)) : yc * ss_silu(zc) * inv * weight[c0 + c];
+    ss_store(out, out_dtype, row * width + c0 + c, v);
   }
 }
 
@@ -492,16 +497,21 @@ TIB_API int tib_ssd_scan(const void* xbc, int xbc_dtype, int64_t ld_xbc, const v
 #undef TIB_SCAN_CASE
 }
 
-// y: [rows, width] fp32; z: rows of z_dtype (row stride ldz, first column z_col); weight [width] fp32; out [rows, width].
+// y: [rows, width] fp32; z: rows of z_dtype (row stride ldz, first column z_col); weight [width] fp32; out [rows, width];
+// gate_last: the norm of y, times sigmoid(z), instead of the norm of y * silu(z).
 TIB_API int tib_gated_group_norm(const float* y, const void* z, int z_dtype, int64_t ldz, int z_col, const float* weight, float eps,
-                                 void* out, int out_dtype, int rows, int width, int parts, cudaStream_t stream) {
+                                 void* out, int out_dtype, int rows, int width, int parts, int gate_last, cudaStream_t stream) {
   if (rows == 0 || width == 0) return TIB_OK;
   if (!y || !z || !weight || !out || rows < 0) return TIB_E_ARG;
   if (parts < 1 || width % parts || parts > 65535) return TIB_E_SIZE;
   if (!ss_known(z_dtype) || !ss_known(out_dtype)) return TIB_E_DTYPE;
   const int part = width / parts;
   const int threads = part >= 1024 ? 256 : part >= 256 ? 128 : 64;
-  TIB_LAUNCH_DEPENDENT(gated_group_norm_kernel, dim3(rows, parts), threads, 0, stream, y, z, z_dtype, ldz, z_col, weight, eps, out,
-                       out_dtype, width, part);
+  if (gate_last)
+    TIB_LAUNCH_DEPENDENT(gated_group_norm_kernel<true>, dim3(rows, parts), threads, 0, stream, y, z, z_dtype, ldz, z_col, weight,
+                         eps, out, out_dtype, width, part);
+  else
+    TIB_LAUNCH_DEPENDENT(gated_group_norm_kernel<false>, dim3(rows, parts), threads, 0, stream, y, z, z_dtype, ldz, z_col, weight,
+                         eps, out, out_dtype, width, part);
   return TIB_OK;
 }

@@ -120,7 +120,7 @@ def lib() -> ctypes.CDLL:
                    "tib_gemm_tcgen05", "tib_gemm_tcgen05_supports",
                    "tib_gemm_tcgen05_swapab", "tib_gemm_tcgen05_swapab_supports", "tib_gemm_decode", "tib_gemm_decode_supports",
                    "tib_plan_attention", "tib_plan_product", "tib_blas_gemm_batched",
-                   "tib_add_pair", "tib_unit_norm_add", "tib_sigmoid_gate", "tib_gelu_gate_table", "tib_relu_squared",
+                   "tib_add_pair", "tib_unit_norm_add", "tib_sigmoid_gate", "tib_gelu_gate_table", "tib_relu_squared", "tib_gelu",
                    "tib_scale_f32", "tib_pair_rows", "tib_add_vector", "tib_linear_attention", "tib_linear_attention_chunk",
                    "tib_latent_append", "tib_latent_attention", "tib_latent_attention_splits", "tib_moe_route", "tib_moe_group", "tib_router_logits",
                    "tib_moe_expert_product", "tib_moe_combine", "tib_glu_clamp", "tib_layernorm", "tib_layernorm_tail",
@@ -130,7 +130,8 @@ def lib() -> ctypes.CDLL:
                    "tib_pooled_window_attention_splits", "tib_pooled_window_attention_part_floats",
                    "tib_input_conv", "tib_norm_conv_step", "tib_row_norm_append", "tib_talking_heads_attention",
                    "tib_talking_heads_takes_mma", "tib_talking_heads_takes_step", "tib_talking_heads_key_span",
-                   "tib_talking_heads_tiles_per_part"):
+                   "tib_talking_heads_tiles_per_part", "tib_conv_norm_append", "tib_matrix_memory", "tib_matrix_memory_tile",
+                   "tib_matrix_memory_chunk", "tib_matrix_memory_max_dim", "tib_matrix_memory_takes_chunks"):
             getattr(library, fn).restype = c_int
         _signatures_set = True
     return library
@@ -756,15 +757,22 @@ def add_pair(residual: torch.Tensor, a: torch.Tensor, b: torch.Tensor | None = N
     return residual
 
 
-def unit_norm_add(residual: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float) -> torch.Tensor:
-    """residual += y / sqrt(mean(y^2) + eps) * weight, statistics and sum in fp32."""
+def unit_norm_add(residual: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float, scale: float = 1.0,
+                  copy: torch.Tensor | None = None) -> torch.Tensor:
+    """residual += scale * (y / sqrt(mean(y^2) + eps) * weight), statistics and sum in fp32; ``copy`` (if given) gets the new
+    rows in its own type."""
     _need(residual, "residual", torch.float32), _need(weight, "weight", torch.float32)
     n, width = residual.shape
     _rows_of(y, "y", width)
     if y.shape[0] != n or weight.numel() != width:
         raise KernelError("unit_norm_add: shapes do not fit")
+    if copy is not None:
+        _need(copy, "copy")
+        if copy.shape != residual.shape:
+            raise KernelError("unit_norm_add: copy does not fit")
     _check("unit_norm_add", lib().tib_unit_norm_add(_ptr(residual), _ptr(y), c_int(_code(y.dtype)), c_int64(y.stride(0)),
-                                                    _ptr(weight), c_int(n), c_int(width), c_float(eps), _stream()))
+                                                    _ptr(weight), c_int(n), c_int(width), c_float(eps), c_float(scale),
+                                                    _ptr(copy), c_int(_code(copy.dtype) if copy is not None else 0), _stream()))
     return residual
 
 
@@ -809,6 +817,15 @@ def relu_squared(x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
         raise KernelError("relu_squared: sizes differ")
     _check("relu_squared", lib().tib_relu_squared(_ptr(x), c_int(_code(x.dtype)), _ptr(out), c_int(_code(out.dtype)),
                                                   c_int64(x.numel()), _stream()))
+    return out
+
+
+def gelu(x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """out = x * Phi(x) element by element (the erf form of gelu), in fp32."""
+    _need(x, "x"), _need(out, "out")
+    if x.numel() != out.numel():
+        raise KernelError("gelu: sizes differ")
+    _check("gelu", lib().tib_gelu(_ptr(x), c_int(_code(x.dtype)), _ptr(out), c_int(_code(out.dtype)), c_int64(x.numel()), _stream()))
     return out
 
 
@@ -926,11 +943,11 @@ def latent_append(dkv: torch.Tensor, q: torch.Tensor, folded: torch.Tensor, keys
 def latent_attention(folded: torch.Tensor, keys: torch.Tensor, out: torch.Tensor, q_start: torch.Tensor, kv_start: torch.Tensor,
                      slots: torch.Tensor, block_table: torch.Tensor, n_entries: int, max_q_len: int, heads: int, rank: int,
                      rot: int, scale: float, error_word: torch.Tensor | None = None, max_kv_len: int = 0,
-                     force_simt: bool = False) -> torch.Tensor:
+                     force_simt: bool = False, sink: torch.Tensor | None = None) -> torch.Tensor:
     """Causal attention of folded queries [tokens, heads, rank + rot] (fp32) over paged latent rows; the value of a
     key is its first ``rank`` elements.  ``out``: [tokens, heads, rank] fp32.  A step of single tokens only
     (``max_q_len`` 1) that names the longest context (``max_kv_len``) cuts every context into runs that go to blocks of
-    their own and are merged by a second kernel."""
+    their own and are merged by a second kernel.  ``sink`` [heads] fp32: exp(sink) is added to the softmax's denominator."""
     _need(folded, "folded", torch.float32), _need(out, "out", torch.float32)
     for name, t in (("q_start", q_start), ("kv_start", kv_start), ("slots", slots), ("block_table", block_table)):
         _need(t, name, torch.int32)
@@ -941,6 +958,10 @@ def latent_attention(folded: torch.Tensor, keys: torch.Tensor, out: torch.Tensor
         raise KernelError(f"latent_attention: pages of shape {tuple(keys.shape)} do not fit")
     if q_start.numel() < n_entries + 1 or kv_start.numel() < n_entries or slots.numel() < n_entries:
         raise KernelError("latent_attention: entry arrays are shorter than n_entries")
+    if sink is not None:
+        _need(sink, "sink", torch.float32)
+        if sink.numel() != heads:
+            raise KernelError("latent_attention: sink holds one number per head")
     splits, partial = 1, None
     if max_q_len == 1 and max_kv_len > 0 and n == n_entries:
         splits = int(lib().tib_latent_attention_splits(c_int(n_entries), c_int(heads), c_int(max_kv_len)))
@@ -949,7 +970,7 @@ def latent_attention(folded: torch.Tensor, keys: torch.Tensor, out: torch.Tensor
     _check("latent_attention", lib().tib_latent_attention(
         _ptr(folded), _ptr(keys), _ptr(out), _ptr(q_start), _ptr(kv_start), _ptr(slots), _ptr(block_table),
         c_int(block_table.stride(0)), c_int(n_entries), c_int(max_q_len), c_int(heads), c_int(rank), c_int(rot),
-        c_int(keys.shape[2]), c_int64(keys.stride(0)), c_int(keys.shape[0]), c_float(scale), _ptr(partial), c_int(splits),
+        c_int(keys.shape[2]), c_int64(keys.stride(0)), c_int(keys.shape[0]), c_float(scale), _ptr(sink), _ptr(partial), c_int(splits),
         c_int(max_kv_len), c_int(int(force_simt)), _ptr(error_word), c_int(_code(keys.dtype)), _stream()))
     if partial is not None:
         count_launches(1)
@@ -957,16 +978,20 @@ def latent_attention(folded: torch.Tensor, keys: torch.Tensor, out: torch.Tensor
 
 
 # ---------------------------------------------------------------------------
-MOE_ACT = {"none": 0, "relu2": 1, "silu": 2, "glu_clamp": 3, "swiglu": 4}
+MOE_ACT = {"none": 0, "relu2": 1, "silu": 2, "glu_clamp": 3, "swiglu": 4, "gelu": 5}
 MOE_GATED = ("glu_clamp", "swiglu")      # activations over (gate, up) row pairs: half as many columns leave
 
 
-def router_logits(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-    """out[t, e] = x[t] . w[e] in fp32, for a few rows ``w`` (fp32): every sum in an order fixed by k alone."""
+def router_logits(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: torch.Tensor | None = None) -> torch.Tensor:
+    """out[t, e] = x[t] . w[e] (+ bias[e]) in fp32, for a few rows ``w`` (fp32): every sum in an order fixed by k alone."""
     _rows_of(x, "x"), _need(w, "w", torch.float32), _rows_of(out, "out")
     if out.dtype != torch.float32 or w.dim() != 2 or x.shape[1] != w.shape[1] or out.shape != (x.shape[0], w.shape[0]):
         raise KernelError("router_logits: shapes or types do not fit")
-    _check("router_logits", lib().tib_router_logits(_ptr(x), c_int(_code(x.dtype)), c_int64(x.stride(0)), _ptr(w), _ptr(out),
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+        if bias.numel() != w.shape[0]:
+            raise KernelError("router_logits: the bias holds one number per row")
+    _check("router_logits", lib().tib_router_logits(_ptr(x), c_int(_code(x.dtype)), c_int64(x.stride(0)), _ptr(w), _ptr(bias), _ptr(out),
                                                     c_int64(out.stride(0)), c_int(x.shape[0]), c_int(w.shape[0]), c_int(x.shape[1]),
                                                     _stream()))
     return out
@@ -1330,16 +1355,17 @@ def ssd_scan(xbc: torch.Tensor, dt_rows: torch.Tensor, dt_col: int, dt_bias: tor
 
 
 def gated_group_norm(y: torch.Tensor, z_rows: torch.Tensor, z_col: int, weight: torch.Tensor, eps: float, out: torch.Tensor,
-                     parts: int) -> torch.Tensor:
+                     parts: int, gate_last: bool = False) -> torch.Tensor:
     """out = v / sqrt(mean(v^2) + eps) * weight with v = y * silu(z) and the mean taken over each of ``parts`` equal runs
-    of the row; y fp32, z = ``z_rows[:, z_col : z_col + width]``."""
+    of the row; y fp32, z = ``z_rows[:, z_col : z_col + width]``.  ``gate_last``: v = y, and the result is multiplied by
+    sigmoid(z)."""
     _need(y, "y", torch.float32), _rows_of(z_rows, "z_rows"), _need(weight, "weight", torch.float32), _need(out, "out")
     n, width = y.shape
     if out.shape != y.shape or weight.numel() != width or z_rows.shape[0] != n or z_col < 0 or z_col + width > z_rows.shape[1]:
         raise KernelError("gated_group_norm: shapes do not fit")
     _check("gated_group_norm", lib().tib_gated_group_norm(
         _ptr(y), _ptr(z_rows), c_int(_code(z_rows.dtype)), c_int64(z_rows.stride(0)), c_int(z_col), _ptr(weight), c_float(eps),
-        _ptr(out), c_int(_code(out.dtype)), c_int(n), c_int(width), c_int(parts), _stream()))
+        _ptr(out), c_int(_code(out.dtype)), c_int(n), c_int(width), c_int(parts), c_int(int(gate_last)), _stream()))
     return out
 
 
@@ -1402,7 +1428,7 @@ def pool_blocks(keys: torch.Tensor, values: torch.Tensor, block_table: torch.Ten
 def pooled_window_attention(q: torch.Tensor, out: torch.Tensor, q_start: torch.Tensor, kv_start: torch.Tensor, slots: torch.Tensor,
                             keys: torch.Tensor, values: torch.Tensor, block_table: torch.Tensor, block_keys: torch.Tensor | None,
                             block_values: torch.Tensor | None, block_block_table: torch.Tensor | None, n_entries: int,
-                            max_q_len: int, heads: int, kv_heads: int, *, window: int, pool: int, scale: float,
+                            max_q_len: int, heads: int, kv_heads: int, *, window: int, pool: int, scale: float, keep: int = 0,
                             temp: torch.Tensor | None = None, sink: torch.Tensor | None = None,
                             value_freq: torch.Tensor | None = None, gate: torch.Tensor | None = None,
                             error_word: torch.Tensor | None = None, force_simt: bool = False,
@@ -1411,8 +1437,9 @@ def pooled_window_attention(q: torch.Tensor, out: torch.Tensor, q_start: torch.T
     with 0 <= i - j < window and the blocks b of ``pool`` positions with b * pool + pool - 1 <= i - window (their means K_b,
     V_b from the strided pages), scores q . k * scale * temp[h], exp(sink[h]) added to the denominator; turn_back undoes at
     position i the rotation the values were cached with (``value_freq``; None: none).  ``pool`` 0: the window alone.
+    ``keep`` > 0: the first ``keep`` tokens of a sequence are seen from behind the window too (without blocks and ``rel_bias``).
     ``rel_bias`` [heads, span] fp32: rel_bias[h, min(i - j, span - 1)] is added to the score of token j (as it is: neither
-    ``scale`` nor ``temp`` multiplies it).  A step of single tokens only on the tensor cores (no turned values, no gate) that
+    ``scale`` nor ``temp`` multiplies it).  A step of single tokens only on the tensor cores (no turned values) that
     names the longest context (``max_kv_len``) shares every context's visible keys out over ``splits`` blocks (None: enough
     to fill the GPU) whose sums a second small kernel adds in a fixed order.
     bfloat16 steps run on the tensor cores when the head sizes are multiples of 8 up to 128, unless ``force_simt``."""
@@ -1443,10 +1470,10 @@ def pooled_window_attention(q: torch.Tensor, out: torch.Tensor, q_start: torch.T
             raise KernelError("pooled_window_attention: rel_bias must be [heads, span]")
     partial, n_splits = None, 1
     if (max_q_len == 1 and n == n_entries and max_kv_len > 0 and q.dtype == torch.bfloat16 and not force_simt
-            and value_freq is None and gate is None and dim % 8 == 0 and vdim % 8 == 0 and dim <= 128 and vdim <= 128
+            and value_freq is None and dim % 8 == 0 and vdim % 8 == 0 and dim <= 128 and vdim <= 128
             and heads // kv_heads <= 16):
         n_splits = splits if splits is not None else int(lib().tib_pooled_window_attention_splits(
-            c_int(n_entries), c_int(heads), c_int(kv_heads), c_int(min(window, max_kv_len) + (max_kv_len // pool if pool else 0))))
+            c_int(n_entries), c_int(heads), c_int(kv_heads), c_int(min(window + keep, max_kv_len) + (max_kv_len // pool if pool else 0))))
         if n_splits > 1:
             floats = int(lib().tib_pooled_window_attention_part_floats(c_int(vdim)))
             partial = torch.empty((n_splits, n, heads, floats), dtype=torch.float32, device=q.device)
@@ -1458,7 +1485,7 @@ def pooled_window_attention(q: torch.Tensor, out: torch.Tensor, q_start: torch.T
         c_int(block_table.stride(0)), c_int(page_size), c_int64(page_stride), c_int(num_pages),
         _ptr(block_keys if pool > 0 else None), _ptr(block_values if pool > 0 else None),
         _ptr(block_block_table if pool > 0 else None), c_int(b_table_stride), c_int(b_page_size), c_int64(b_stride), c_int(b_pages),
-        c_int(n_entries), c_int(max_q_len), c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim), c_int(window), c_int(pool),
+        c_int(n_entries), c_int(max_q_len), c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim), c_int(window), c_int(keep), c_int(pool),
         c_float(scale), _ptr(temp), _ptr(sink), _ptr(value_freq), _ptr(gate), c_int(_code(gate.dtype) if gate is not None else 0),
         c_int64(ld_gate), _ptr(rel_bias), c_int(rel_bias.shape[1] if rel_bias is not None else 0), _ptr(partial),
         c_int(n_splits), c_int(n), _ptr(error_word), c_int(_code(q.dtype)), c_int(int(force_simt)), _stream()))
@@ -1686,4 +1713,123 @@ def talking_heads_attention(q: torch.Tensor, out: torch.Tensor, q_start: torch.T
     for first in range(0, n, chunk):
         count_launches(2)
         call(1, first=first, last=min(n, first + chunk), scores=scores, lse=lse, key_span=key_span)
+    return out
+
+
+# ---------------------------------------------------------------------------
+# Queries and keys that pass a short convolution ahead of norm and rotation (csrc/conv_norm_append.cu).
+def conv_norm_append(proj: torch.Tensor, q_off: int, k_off: int, q_out: torch.Tensor, keys: torch.Tensor, values: torch.Tensor,
+                     q_conv: torch.Tensor, k_conv: torch.Tensor, positions: torch.Tensor, block_table: torch.Tensor,
+                     q_start: torch.Tensor, slots: torch.Tensor, n_entries: int, heads: int, kv_heads: int, dim: int, *,
+                     freq: torch.Tensor, q_weight: torch.Tensor | None = None, k_weight: torch.Tensor | None = None, eps: float = 1e-6,
+                     state: torch.Tensor | None = None, state_off: int = 0, error_word: torch.Tensor | None = None) -> torch.Tensor:
+    """Per channel of the q and k columns of ``proj``, y_t = sum_j conv[j] * u_(t - taps + 1 + j) within each entry (``q_conv`` /
+    ``k_conv``: [taps, columns] fp32; the rows ahead of an entry come from ``state[slot, state_off:]``, laid out [taps - 1, q
+    columns + k columns], where the entry's last rows are then left).  The convolved k rows go to the pages of ``values`` as
+    they are; both rows are divided by their root mean square and multiplied by a weight per element (weights None: not), the
+    pairs (2i, 2i + 1) of the first 2 * len(freq) elements of every head are turned by position * freq[i], and q goes to
+    ``q_out``, k to the pages of ``keys``."""
+    _rows_of(proj, "proj"), _need(q_out, "q_out", proj.dtype), _need(freq, "freq", torch.float32)
+    for name, t in (("positions", positions), ("block_table", block_table), ("q_start", q_start), ("slots", slots)):
+        _need(t, name, torch.int32)
+    n = proj.shape[0]
+    taps = q_conv.shape[0]
+    for name, t, width in (("q_conv", q_conv, heads * dim), ("k_conv", k_conv, kv_heads * dim)):
+        _need(t, name, torch.float32)
+        if t.shape != (taps, width):
+            raise KernelError(f"conv_norm_append: {name} does not fit")
+    for t, width in ((q_weight, heads * dim), (k_weight, kv_heads * dim)):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != width or not t.is_contiguous()):
+            raise KernelError("conv_norm_append: a weight does not fit")
+    if q_out.shape != (n, heads * dim) or keys.dtype != proj.dtype or max(q_off + heads * dim, k_off + kv_heads * dim) > proj.shape[1]:
+        raise KernelError("conv_norm_append: shapes or types do not fit")
+    if q_start.numel() < n_entries + 1 or slots.numel() < n_entries or positions.numel() < n:
+        raise KernelError("conv_norm_append: the batch's arrays are too short")
+    stride = 0
+    if taps > 1:
+        if state is None:
+            raise KernelError("conv_norm_append: a convolution of several taps needs its state")
+        _need(state, "state", torch.float32)
+        if state.dim() != 2 or state_off < 0 or state_off + (taps - 1) * (heads + kv_heads) * dim > state.shape[1]:
+            raise KernelError("conv_norm_append: the state does not fit")
+        stride = state.stride(0)
+    num_pages, page_size, page_stride = _pages(keys, values, kv_heads, dim, dim, "conv_norm_append")
+    _check("conv_norm_append", lib().tib_conv_norm_append(
+        _ptr(proj), c_int64(proj.stride(0)), c_int(q_off), c_int(k_off), _ptr(q_conv), _ptr(k_conv), c_int(taps), _ptr(q_weight),
+        _ptr(k_weight), c_float(eps), _ptr(freq), c_int(freq.numel()), _ptr(q_out), _ptr(keys), _ptr(values), _ptr(positions),
+        _ptr(block_table), c_int(block_table.stride(0)), _ptr(q_start), _ptr(slots), c_int(n_entries), _ptr(state if taps > 1 else None),
+        c_int64(stride), c_int64(state_off), c_int(n), c_int(heads), c_int(kv_heads), c_int(dim), c_int(page_size),
+        c_int64(page_stride), c_int(num_pages), _ptr(error_word), c_int(_code(proj.dtype)), _stream()))
+    return q_out
+
+
+# ---------------------------------------------------------------------------
+# The matrix memory with exponential gates (csrc/matrix_memory.cu).
+def matrix_memory_max_dim() -> int:
+    """The largest key width of a head the kernels take."""
+    return int(lib().tib_matrix_memory_max_dim())
+
+
+MATRIX_MEMORY_TILE = 128      # value columns of a tile (checked against the library at the first call)
+MATRIX_MEMORY_WALK = 8        # portions up to this long are walked token by token, longer ones cut into chunks where the shapes allow
+
+
+def matrix_memory_state_floats(heads: int, dim: int, vdim: int) -> int:
+    """Floats of state a request holds: S of every head, then n and m per head and tile of value columns (a multiple of 4)."""
+    tiles = -(-vdim // MATRIX_MEMORY_TILE)
+    return -(-heads * (dim * vdim + tiles * (dim + 1)) // 4) * 4
+
+
+def matrix_memory(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int, x: torch.Tensor, gate_weight: torch.Tensor,
+                  gate_bias: torch.Tensor, cap: float, state: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, n_entries: int,
+                  max_q_len: int, norm_weight: torch.Tensor, eps: float, out: torch.Tensor, *, heads: int, dim: int, vdim: int,
+                  q_scale: float, walk: bool | None = None) -> torch.Tensor:
+    """Per head, with i = cap tanh((w_i . x + b_i) / cap), f = logsigmoid(cap tanh((w_f . x + b_f) / cap)) and m_t = max(f + m, i):
+    S_t = exp(f + m - m_t) S + exp(i - m_t) k v^T, n_t likewise with k alone, y = S_t^T q / (max(|n_t . q|, exp(-m_t)) + 1e-6);
+    out = y / rms(y) * norm_weight * sigmoid(gate).  ``proj`` holds q, k, v and the gate's logits at their columns (q is multiplied by
+    ``q_scale``); ``gate_weight`` [2 * heads, width] (i of every head, then f) and ``gate_bias`` are fp32, ``x`` the input rows they
+    multiply; ``state`` [slots, floats] is read and left updated.  ``walk``: token by token (None: decided by the portions' length
+    and the shapes)."""
+    _rows_of(proj, "proj"), _rows_of(x, "x"), _need(state, "state", torch.float32), _need(out, "out", proj.dtype)
+    for name, t in (("gate_weight", gate_weight), ("gate_bias", gate_bias), ("norm_weight", norm_weight)):
+        _need(t, name, torch.float32)
+    _need(q_start, "q_start", torch.int32), _need(slots, "slots", torch.int32)
+    n, dev = proj.shape[0], proj.device
+    library = lib()
+    if int(library.tib_matrix_memory_tile()) != MATRIX_MEMORY_TILE:
+        raise KernelError("matrix_memory: the library's tile differs")
+    if (x.shape[0] != n or x.dtype != proj.dtype or gate_weight.shape != (2 * heads, x.shape[1]) or gate_bias.numel() != 2 * heads
+            or norm_weight.numel() != heads * vdim or out.shape != (n, heads * vdim) or state.dim() != 2
+            or state.shape[1] < matrix_memory_state_floats(heads, dim, vdim)
+            or max(q_off + heads * dim, k_off + heads * dim, v_off + heads * vdim, g_off + heads * vdim) > proj.shape[1]):
+        raise KernelError("matrix_memory: shapes or types do not fit")
+    if q_start.numel() < n_entries + 1 or slots.numel() < n_entries:
+        raise KernelError("matrix_memory: entry arrays are shorter than n_entries")
+    takes_chunks = proj.dtype == torch.bfloat16 and bool(library.tib_matrix_memory_takes_chunks(c_int(dim), c_int(vdim)))
+    chunks = takes_chunks and max_q_len > MATRIX_MEMORY_WALK if walk is None else not walk
+    logits = None
+    if max_q_len > 1:      # (a step of single tokens works its gate rows out in the same launch)
+        logits = router_logits(x, gate_weight, torch.empty((n, 2 * heads), dtype=torch.float32, device=dev))
+    fused = vdim <= MATRIX_MEMORY_TILE
+    y = None if fused else torch.empty((n, heads * vdim), dtype=torch.float32, device=dev)
+    cum = log_in = top = top0 = run_state = run_n = run_keep = None
+    capacity = 0
+    if chunks:
+        capacity = n // int(library.tib_matrix_memory_chunk()) + n_entries
+        cum = torch.empty((heads, n), dtype=torch.float64, device=dev)
+        log_in, top = (torch.empty((heads, n), dtype=torch.float32, device=dev) for _ in range(2))
+        top0 = torch.empty((heads, n_entries), dtype=torch.float32, device=dev)
+        run_state = torch.empty((capacity, heads, dim, vdim), dtype=torch.float32, device=dev)
+        run_n = torch.empty((capacity, heads, dim), dtype=torch.float32, device=dev)
+        run_keep = torch.empty((capacity, heads), dtype=torch.float32, device=dev)
+        count_launches(3)
+    _check("matrix_memory", library.tib_matrix_memory(
+        _ptr(proj), c_int64(proj.stride(0)), c_int(q_off), c_int(k_off), c_int(v_off), c_int(g_off), c_float(q_scale), _ptr(logits),
+        _ptr(x), c_int64(x.stride(0)), _ptr(gate_weight), c_int(x.shape[1]), _ptr(gate_bias), c_float(cap), _ptr(state),
+        c_int64(state.stride(0)), _ptr(q_start), _ptr(slots), _ptr(norm_weight if fused else None), c_float(eps), _ptr(y),
+        _ptr(out if fused else None), c_int(heads), c_int(dim), c_int(vdim), c_int(n_entries), c_int(n), c_int(max_q_len),
+        c_int(int(chunks)), _ptr(cum), _ptr(log_in), _ptr(top), _ptr(top0), _ptr(run_state), _ptr(run_n), _ptr(run_keep),
+        c_int64(capacity), c_int(_code(proj.dtype)), _stream()))
+    if not fused:
+        gated_group_norm(y, proj, g_off, norm_weight, eps, out, heads, gate_last=True)
     return out

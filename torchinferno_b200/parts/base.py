@@ -63,12 +63,15 @@ class CacheSpec:
     ``stride``: s > 1 means the cache holds one entry for every full run of s tokens (entry b stands for the
     positions b*s .. b*s + s - 1 and exists once the last of them has arrived): a summary of the run, such as
     the mean of its keys.  Such a cache grows s times slower than the request.
+
+    ``keep_first``: with a window, the tokens 0 .. keep_first - 1 stay readable from behind it, so their pages are kept.
     """
     kv_heads: int
     head_dim: int
     window: int | None = None
     value_dim: int | None = None
     stride: int = 1
+    keep_first: int = 0
 
     @property
     def value_width(self) -> int:
@@ -195,6 +198,16 @@ class ResidualStream:
                 self.pending = None
         return out
 
+    def rows(self) -> torch.Tensor:
+        """The residual itself in the activation type, for a sublayer that reads it without a norm."""
+        residual = self.settle()
+        if self.dtype == torch.float32:
+            return residual
+        if self.activation_copy is None:
+            from torchinferno_b200.kernels import ops
+            self.activation_copy = ops.cast(residual, torch.empty(residual.shape, dtype=self.dtype, device=residual.device))
+        return self.activation_copy
+
     def add(self, delta: torch.Tensor) -> None:
         if self.pending is not None:
             raise RuntimeError("a delta is already pending; a norm must fold it in first")
@@ -207,6 +220,7 @@ class ResidualStream:
             from torchinferno_b200.kernels import ops
             ops.add_pair(self.residual, self.pending)
             self.pending = None
+            self.activation_copy = None
         return self.residual
 
 
@@ -352,6 +366,6 @@ def _ensure_builtin() -> None:
         return
     _loaded = True
     from torchinferno_b200.parts import (attention, biased_attention, block, gated_recurrence, hyper_block,  # noqa: F401
-                                         input_stages, latent_attention, linear_attention, mlp, moe, norm, parallel_block,
-                                         pooled_window_attention, rope, sandwich_block, sigmoid_attention, state_space,
+                                         input_stages, kept_window_attention, latent_attention, linear_attention, matrix_memory,
+                                         mlp, moe, norm, parallel_block, pooled_window_attention, postnorm_block, rope, sandwich_block, sigmoid_attention, state_space,
                                          stream_stages, talking_heads_attention)

@@ -3,7 +3,8 @@
 From the layer input x: q = W_q x, laid out head by head as [``dim`` unrotated ; ``rot_dim`` rotated]; W_dkv x has
 ``kv_rank + rot_dim`` rows, the first kv_rank RMS-normed (plain weight) are the latent c, the last rot_dim, rotated,
 are a key part r that all heads share.  Head j's key is [W_uk_j c ; r] and its value W_uv_j c; causal softmax with
-the given scale; the heads' outputs are optionally multiplied by sigmoid(W_g x), element by element (``gate=True``) or
+the given scale (with ``sink`` a learned number per head, ``sink_name``, whose exponential is added to the softmax's denominator:
+it has neither key nor value); the heads' outputs are optionally multiplied by sigmoid(W_g x), element by element (``gate=True``) or
 with one gate per head (``gate="head"``, W_g has ``heads`` rows), then projected by W_o.  With ``q_rank`` the queries are
 made in two steps: the rows W_dq x of that width, RMS-normed and multiplied by a weight, then W_uq on the result.
 
@@ -28,11 +29,11 @@ from torchinferno_b200.parts.base import CacheSpec, LayerContext, Mixer, WeightS
 
 class LatentAttention(Mixer):
     def __init__(self, *, hidden_size: int, heads: int, dim: int, rot_dim: int, value_dim: int, kv_rank: int, scale: float,
-                 rot_base: float, rot_dims: int | None = None, eps: float = 1e-6, gate: bool | str = True,
+                 rot_base: float, rot_dims: int | None = None, eps: float = 1e-6, gate: bool | str = True, sink: bool = False,
                  q_rank: int | None = None, pairing: str = "interleaved",
                  q_name: str = "q", dkv_name: str = "dkv", latent_norm_name: str = "dkv.norm", uk_name: str = "uk",
                  uv_name: str = "uv", g_name: str = "g", o_name: str = "o", dq_name: str = "dq", q_norm_name: str = "dq.norm",
-                 uq_name: str = "uq", dtype: torch.dtype, device: torch.device) -> None:
+                 uq_name: str = "uq", sink_name: str = "sink", dtype: torch.dtype, device: torch.device) -> None:
         super().__init__(dtype=dtype, device=device)
         if gate not in (True, False, "element", "head") or pairing not in ("interleaved", "half"):
             raise ValueError(f"unknown gate {gate!r} or pairing {pairing!r}")
@@ -47,7 +48,9 @@ class LatentAttention(Mixer):
         self.inv_freq = (torch.tensor(float(rot_base), dtype=torch.float64) ** (-2.0 * i / max(self.rot_dims, 1))) \
             .to(torch.float32).to(device)
         self.names = {"q": q_name, "dkv": dkv_name, "norm": latent_norm_name, "uk": uk_name, "uv": uv_name, "g": g_name,
-                      "o": o_name, "dq": dq_name, "q_norm": q_norm_name, "uq": uq_name}
+                      "o": o_name, "dq": dq_name, "q_norm": q_norm_name, "uq": uq_name, "sink": sink_name}
+        self.has_sink = bool(sink)
+        self.sink: torch.Tensor | None = None
         self.in_weight: LinearWeight | None = None
         self.uq_weight: LinearWeight | None = None
         self.o_weight: LinearWeight | None = None
@@ -65,6 +68,8 @@ class LatentAttention(Mixer):
                  WeightSpec(n["norm"], (self.kv_rank,), init="ones", role="vector"),
                  WeightSpec(n["uk"], (h * self.dim, self.kv_rank), std=rank_std),
                  WeightSpec(n["uv"], (h * self.value_dim, self.kv_rank), std=rank_std)]
+        if self.has_sink:
+            specs.append(WeightSpec(n["sink"], (h,), std=1.0, role="vector"))
         if self.gate:
             specs.append(WeightSpec(n["g"], (h if self.gate_per_head else h * self.value_dim, w), std=std))
         specs.append(WeightSpec(n["o"], (w, h * self.value_dim), std=(h * self.value_dim) ** -0.5))
@@ -82,6 +87,8 @@ class LatentAttention(Mixer):
             self.q_norm_weight = weights[n["q_norm"]].to(torch.float32).contiguous()
         self.o_weight = LinearWeight(weights[n["o"]], few_rows_tcgen05=None)
         self.latent_norm_weight = weights[n["norm"]].to(torch.float32).contiguous()
+        if self.has_sink:
+            self.sink = weights[n["sink"]].to(torch.float32).contiguous()
         uk = weights[n["uk"]].view(h, self.dim, self.kv_rank)              # per head [in = dim, out = kv_rank]
         self.uv_weight = weights[n["uv"]].view(h, self.value_dim, self.kv_rank).contiguous()   # per head [out, in]
         if uk.dtype == torch.float32:
@@ -116,7 +123,8 @@ class LatentAttention(Mixer):
             ops.library_gemm_batched(q_plain, self.uk_weight, folded[:, :, :c], w_kn=True)
         latent_out = torch.empty((n, h, c), dtype=torch.float32, device=x.device)
         ops.latent_attention(folded, kv.keys, latent_out, batch.q_start, batch.kv_start, batch.slots, kv.block_table,
-                             batch.n_entries, batch.max_q_len, h, c, r, self.scale, ctx.error_word, max_kv_len=batch.max_kv_len)
+                             batch.n_entries, batch.max_q_len, h, c, r, self.scale, ctx.error_word, max_kv_len=batch.max_kv_len,
+                             sink=self.sink)
         heads_out = torch.empty((n, h, self.value_dim), dtype=x.dtype, device=x.device)
         if x.dtype == torch.float32:
             for j in range(h):

@@ -12,6 +12,9 @@ as one product over row pairs (gate i, up i).  ``weight_on_input``: the router w
 instead of its output, sum of expert(w x); it is applied to the 32-bit sums of the first product, ahead of the clamps
 (W (w x) = w (W x)), so the input rows are not rounded a second time.
 
+``activation="gelu"``: the expert is W_down gelu(W_up x) with the erf form of gelu.  ``router_bias``: a tensor of one number per
+router output (the router's name with ``.b`` added) is part of its logits.
+
 ``activation="swiglu"``: an expert is the plain gated unit W_down (silu(W_gate x) * (W_up x)), gate and up again as row
 pairs of one product.
 
@@ -42,13 +45,13 @@ class RoutedExperts(FeedForward):
                  down_name: str = "down", shared_prefix: str = "shared.", shared_gate_name: str = "sg", gate_name: str = "gate",
                  limit: float = 0.0, shared_limit: float | None = None, alpha: float = 1.702, weight_on_input: bool = False,
                  identity: int = 0, correction: bool = False, correction_name: str = "correction",
-                 groups: tuple[int, int] | None = None, dtype: torch.dtype, device: torch.device) -> None:
+                 groups: tuple[int, int] | None = None, router_bias: bool = False, bias_suffix: str = ".b", dtype: torch.dtype, device: torch.device) -> None:
         super().__init__(dtype=dtype, device=device)
         self.identity = int(identity)
         self.routed = experts + self.identity          # outputs of the router
         if experts < 1 or self.identity < 0 or not 1 <= top <= self.routed:
             raise ValueError("top must be between 1 and the number of experts (identity ones included)")
-        if activation not in ("relu2", "silu", "glu_clamp", "swiglu") or scores not in ("softmax", "sigmoid"):
+        if activation not in ("relu2", "silu", "gelu", "glu_clamp", "swiglu") or scores not in ("softmax", "sigmoid"):
             raise ValueError(f"unknown activation {activation!r} or scores {scores!r}")
         self.groups = None if groups is None else (int(groups[0]), int(groups[1]))
         if self.groups is not None:
@@ -59,6 +62,8 @@ class RoutedExperts(FeedForward):
             raise ValueError("experts that hand their input through take their weight on the output")
         self.has_correction, self.correction_name = bool(correction), correction_name
         self.correction: torch.Tensor | None = None
+        self.has_router_bias, self.router_bias_name = bool(router_bias), router_name + bias_suffix
+        self.router_bias: torch.Tensor | None = None
         self.hidden_size, self.experts, self.top, self.expert_size = hidden_size, experts, top, expert_size
         self.activation, self.scores, self.normalize, self.norm_eps = activation, scores, bool(normalize), float(norm_eps)
         self.shared_size, self.shared_gate = int(shared_size or 0), bool(shared_gate and shared_size)
@@ -77,6 +82,8 @@ class RoutedExperts(FeedForward):
         router, _, up, down, shared, gate = self.names
         std = self.hidden_size ** -0.5          # (random weights: rows of about unit size from normed input)
         specs = [WeightSpec(router, (self.routed, self.hidden_size), std=2 * std)]
+        if self.has_router_bias:
+            specs.append(WeightSpec(self.router_bias_name, (self.routed,), std=0.3, role="vector"))
         if self.has_correction:
             specs.append(WeightSpec(self.correction_name, (self.routed,), std=0.05, role="vector"))
         for e in range(self.experts):
@@ -97,6 +104,9 @@ class RoutedExperts(FeedForward):
         router, _, up, down, shared, gate = self.names
         rows = [weights[router]] + ([weights[shared + gate]] if self.shared_gate else [])
         self.router_weight = torch.cat(rows, dim=0).to(torch.float32).contiguous()      # (the router is fp32 in both modes)
+        if self.has_router_bias:
+            bias = weights[self.router_bias_name].to(torch.float32)
+            self.router_bias = torch.cat([bias, bias.new_zeros(len(self.router_weight) - self.routed)]).contiguous()      # (none on a gate row)
         if self.has_correction:
             self.correction = weights[self.correction_name].to(torch.float32).contiguous()
         def first(name_of) -> torch.Tensor:
@@ -116,7 +126,7 @@ class RoutedExperts(FeedForward):
     def forward(self, x: torch.Tensor, ctx: LayerContext) -> torch.Tensor:
         n, dev, top = x.shape[0], x.device, self.top
         logits = torch.empty((n, self.router_weight.shape[0]), dtype=torch.float32, device=dev)
-        ops.router_logits(x, self.router_weight, logits)
+        ops.router_logits(x, self.router_weight, logits, self.router_bias)
         ids = torch.empty((n, top), dtype=torch.int32, device=dev)
         weights = torch.empty((n, top), dtype=torch.float32, device=dev)
         count, keep = self.groups if self.groups is not None else (1, 1)
@@ -136,6 +146,8 @@ class RoutedExperts(FeedForward):
             hidden = linear(x, self.shared_up_weight)
             if self.activation == "relu2":
                 ops.relu_squared(hidden, hidden)
+            elif self.activation == "gelu":
+                ops.gelu(hidden, hidden)
             elif self.activation == "glu_clamp":
                 hidden = ops.glu_clamp(hidden, torch.empty((n, self.shared_size), dtype=hidden.dtype, device=dev),
                                        self.shared_limit, self.alpha)

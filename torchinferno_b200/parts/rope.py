@@ -46,14 +46,19 @@ def rotary_amplitude(scaling: Mapping[str, Any] | None) -> float:
     return 1.0
 
 
-def rotary_frequencies(rot_dim: int, theta: float, scaling: Mapping[str, Any] | None = None) -> torch.Tensor:
-    """The fp32 frequency table [rot_dim / 2], on the CPU."""
+def rotary_frequencies(rot_dim: int, theta: float, scaling: Mapping[str, Any] | None = None, exact: bool = False) -> torch.Tensor:
+    """The fp32 frequency table [rot_dim / 2], on the CPU.  ``exact``: made in double precision and rounded once (without a law)."""
     if scaling and scaling.get("rope_type") == "yarn":
         missing = [key for key in ("factor", "original", "fast", "slow") if key not in scaling]
         if missing:
             raise ValueError(f"the yarn law lacks {missing}")
         return yarn_frequencies(rot_dim, float(theta), float(scaling["factor"]), float(scaling["original"]),
                                 float(scaling["fast"]), float(scaling["slow"]))
+    if exact:
+        if scaling:
+            raise ValueError("the exact table has no scaling law")
+        i = torch.arange(rot_dim // 2, dtype=torch.float64)
+        return (torch.tensor(float(theta), dtype=torch.float64) ** (-2.0 * i / max(rot_dim, 1))).to(torch.float32)
     exponent = torch.arange(0, rot_dim, 2, dtype=torch.float32) / rot_dim
     inv_freq = 1.0 / (theta ** exponent)
     if not scaling:
@@ -76,7 +81,7 @@ def rotary_frequencies(rot_dim: int, theta: float, scaling: Mapping[str, Any] | 
 
 class RotaryEncoding(PositionEncoding):
     def __init__(self, *, head_dim: int, theta: float, scaling: Mapping[str, Any] | None = None,
-                 rot_dim: int | None = None, interleaved: bool = False,
+                 rot_dim: int | None = None, interleaved: bool = False, exact: bool = False,
                  dtype: torch.dtype, device: torch.device) -> None:
         super().__init__(dtype=dtype, device=device)
         self.head_dim = int(head_dim)
@@ -84,7 +89,7 @@ class RotaryEncoding(PositionEncoding):
         if self.rot_dim % 2 or self.rot_dim > self.head_dim:
             raise ValueError("rot_dim must be even and at most head_dim")
         self.interleaved = bool(interleaved)
-        self.inv_freq = rotary_frequencies(self.rot_dim, float(theta), scaling).to(device)
+        self.inv_freq = rotary_frequencies(self.rot_dim, float(theta), scaling, exact).to(device)
         # cos and sin are multiplied by this (1 for every law but YaRN's); only kernels that take it as an argument
         # may serve an encoding whose amplitude is not 1
         self.amplitude = rotary_amplitude(scaling)
