@@ -488,10 +488,23 @@ def _design_configs(DESIGN_WIDTH: int, DESIGN_HEADS: int, kv_heads: int, dense_f
     bodopel = {"architecture": "Bodopel", "vocab": DESIGN_VOCAB, "width": DESIGN_WIDTH, "max_positions": 8192, "norm": {"eps": 1e-6},
                "embedding": {"scale": 8.0}, "canon": {"taps": 4}, "loop": {"start": 1, "stop": 3, "times": 1},
                "layers": [{"type": "attention", "mixer": mixed, "mlp": dense} for _ in range(DESIGN_LAYERS)]}
-    return {"zipedra": zipedra, "giforax": giforax, "tibalorn": tibalorn, "vofidra": vofidra, "bodopel": bodopel, "llama": llama}
+    # Tadalorn beside Zipedra (the closest: attention over the same latent, state with matrices of the same size, routed experts of
+    # the same sizes), Tibalorn (attention inside a window of the same size, short convolutions) and the same Llama: a matrix memory, an
+    # attention in a window of 512 that keeps 16 first tokens, one over the latent, and the window attention again
+    memory = {"heads": DESIGN_HEADS, "dim": 128, "vdim": 128, "gate_cap": 15.0}
+    kept = {"heads": DESIGN_HEADS, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "conv": 4,
+            "mask": {"size": 512, "keep_first": 16}, "rot": {"base": 500000.0, "dims": 64}}
+    tadalorn = {"architecture": "Tadalorn", "vocab": DESIGN_VOCAB, "width": DESIGN_WIDTH, "norm": {"eps": 1e-6}, "residual_mult": 0.7,
+                "logit_softcap": 30.0,
+                "layers": [{"type": "mlstm", "mixer": memory, "mlp": dense},
+                           {"type": "attention", "mixer": kept, "mlp": routed},
+                           {"type": "latent_attention", "mixer": latent, "mlp": routed},
+                           {"type": "attention", "mixer": kept, "mlp": dense}]}
+    return {"zipedra": zipedra, "giforax": giforax, "tibalorn": tibalorn, "vofidra": vofidra, "bodopel": bodopel, "tadalorn": tadalorn,
+            "llama": llama}
 
 
-DESIGN_ALSO_BESIDE = {"vofidra": ("zipedra",), "bodopel": ("tibalorn",)}      # the closest design of the package, measured in the same call
+DESIGN_ALSO_BESIDE = {"vofidra": ("zipedra",), "bodopel": ("tibalorn",), "tadalorn": ("zipedra", "tibalorn")}      # the closest design of the package, measured in the same call
 
 
 def run_design(args) -> dict:
@@ -557,6 +570,14 @@ def run_design(args) -> dict:
                                ["pooled-window-attention", "--heads", str(args.design_width // 128), "--kv-heads", str(args.design_width // 256)],
                                ["input-conv", "--hidden", str(args.design_width)],
                                ["state-space", "--heads", str(args.design_width // 32)]),
+                   "tadalorn": (["matrix-memory", "--heads", str(args.design_width // 128), "--hidden", str(args.design_width)],
+                                ["linear-attention", "--heads", str(args.design_width // 128)],
+                                ["kept-window-attention", "--heads", str(args.design_width // 128), "--kv-heads", str(args.design_width // 256)],
+                                ["pooled-window-attention", "--heads", str(args.design_width // 128), "--kv-heads", str(args.design_width // 256)],
+                                ["latent-attention", "--heads", str(args.design_width // 128)],
+                                ["norm-back", "--hidden", str(args.design_width)],
+                                ["state-space", "--heads", str(args.design_width // 32)],
+                                ["expert-product", "--hidden", str(args.design_width), "--expert-size", str(args.design_width // 2)]),
                    "vofidra": (["biased-attention", "--heads", str(args.design_width // 128), "--kv-heads", str(args.design_width // 256)],
                                ["latent-attention", "--heads", str(args.design_width // 128)],
                                ["hyper-streams", "--hidden", str(args.design_width)],
@@ -668,7 +689,7 @@ def main(argv=None) -> int:
     parser.add_argument("--gemm-backend", choices=["auto", "tcgen05", "library"], default="auto")
     parser.add_argument("--workloads", nargs="*", default=list(WORKLOADS), choices=list(WORKLOADS),
                         help="serving workloads of the smaller sizes to add to points")
-    parser.add_argument("--design", choices=["zipedra", "giforax", "tibalorn", "vofidra", "bodopel"], default=None,
+    parser.add_argument("--design", choices=["zipedra", "giforax", "tibalorn", "vofidra", "bodopel", "tadalorn"], default=None,
                         help="instead of the headline run: prefill and decode throughput of this design at layer sizes that "
                              "resemble a real model's, beside the closest Llama, and its kernels against the roofline")
     parser.add_argument("--design-width", type=int, default=DESIGN_WIDTH,

@@ -707,7 +707,7 @@ def test_the_state_of_the_convolution_and_what_is_stored():
     need_gpu()
     from torchinferno_b200.kernels import ops
     for dtype, heads, kv, d, taps, rot, page in ((torch.float32, 3, 1, 7, 4, 4, 4), (torch.bfloat16, 4, 2, 16, 3, 16, 8), (torch.bfloat16, 5, 5, 6, 9, 2, 4),
-                                                 (torch.bfloat16, 40, 20, 128, 4, 64, 16), (torch.float32, 2, 2, 300, 2, 300, 16), (torch.bfloat16, 2, 1, 8, 1, 0, 2)):
+                                                 (torch.bfloat16, 40, 20, 128, 4, 64, 16), (torch.float32, 2, 2, 300, 2, 300, 16), (torch.bfloat16, 2, 1, 8, 1, 0, 2), (torch.bfloat16, 3, 2, 16, 2, 6, 4)):
         g = torch.Generator().manual_seed(d * taps)
         T, qw, kw, pad = 40, heads * d, kv * d, 4
         k_off = -(-qw // 8) * 8
@@ -734,7 +734,7 @@ def test_the_state_of_the_convolution_and_what_is_stored():
             pos = list(range(at, at + n)) + list(range(oat, oat + k))
             q_out, error = torch.empty(n + k, qw, dtype=dtype, device=CUDA), torch.zeros(1, dtype=torch.int32, device=CUDA)
             ops.conv_norm_append(rows, 0, k_off, q_out, keys, values, conv[0].cuda(), conv[1].cuda(), _i32(pos), table,
-                                 _i32(np.cumsum([0] + lens).tolist()), _i32([1, 0][:len(lens)]), len(lens), heads, kv, d, freq=freq.cuda(),
+                                 _i32(np.cumsum([0] + lens).tolist()), _i32([1, 0][:len(lens)]), len(lens), max(lens), heads, kv, d, freq=freq.cuda(),
                                  q_weight=gain[0].cuda(), k_weight=gain[1].cuda(), eps=1e-5, state=state, state_off=pad, error_word=error)
             assert int(error) == 0
             assert (q_out.cpu().double().view(n + k, heads, d) - q_want[pos]).abs().max() <= tol * q_want.abs().max()

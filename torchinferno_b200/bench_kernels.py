@@ -15,6 +15,9 @@
     python -m torchinferno_b200.bench_kernels state-space --tokens 2048 --batch 8
     python -m torchinferno_b200.bench_kernels talking-heads --tokens 2048 --batch 8 --context 2048 --window 512
     python -m torchinferno_b200.bench_kernels input-conv --rows 2048
+    python -m torchinferno_b200.bench_kernels kept-window-attention --tokens 2048 --batch 8 --context 2048 --window 512 --keep 16
+    python -m torchinferno_b200.bench_kernels matrix-memory --tokens 2048 --batch 8
+    python -m torchinferno_b200.bench_kernels norm-back --rows 2048
 
 Each run prints one JSON line per case: microseconds (median of CUDA-event timings, an L2 flush
 between iterations), the bytes or flops the kernel has to move or do, and the fraction of the
@@ -330,6 +333,8 @@ def run_expert_product(args) -> None:
     flops = 2 * t * top * w * ff
     report("expert_product[up, relu^2]", timer(lambda: ops.moe_expert_product(x, up, inner, offsets, order, top, x_by_pair=True, act="relu2")),
            flops=flops, tokens=t, experts=e, top=top, hidden=w, expert_size=ff)
+    report("expert_product[up, gelu]", timer(lambda: ops.moe_expert_product(x, up, inner, offsets, order, top, x_by_pair=True, act="gelu")),
+           flops=flops, tokens=t, experts=e, top=top, hidden=w, expert_size=ff)
     report("expert_product[down]", timer(lambda: ops.moe_expert_product(inner, down, outer, offsets, order, top, x_by_pair=False)),
            flops=flops, tokens=t, experts=e, top=top, hidden=w, expert_size=ff)
     gate_up = (torch.randn(e, 2 * ff, w, device="cuda") * 0.02).to(torch.bfloat16)
@@ -592,6 +597,97 @@ def run_input_conv(args) -> None:
         report("relu_squared", timer(lambda: ops.relu_squared(x, out)), bytes_moved=rows * w * 4, rows=rows, hidden=w)
 
 
+def run_kept_window_attention(args) -> None:
+    """The attention over a window that keeps the first tokens on a prompt of --tokens (flops: both products over the tokens a query
+    sees) and on --batch single tokens at --context (bytes: the keys and values each query sees), with a sink and the output gate;
+    and the launch ahead of it (convolution, norm over the whole row, rotation, store; bytes: projected rows read once, queries,
+    keys and values written)."""
+    h, k, d, page, window, keep, taps = args.heads, args.kv_heads, args.head_dim, args.page_size, args.window, args.keep, args.taps
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device="cuda")
+    timer = Timer(args.iters)
+    seen = lambda p: min(p + 1, window + min(keep, max(0, p + 1 - window)))
+    freq = (10000.0 ** (-torch.arange(d // 4, dtype=torch.float64) * 4 / d)).float().cuda()
+    conv = [torch.randn(taps, w, device="cuda") for w in (h * d, k * d)]
+    gain = [torch.ones(w, device="cuda") for w in (h * d, k * d)]
+    sink = torch.zeros(h, device="cuda")
+    for mode in ("prompt", "single tokens"):
+        n_entries, ctx = (1, args.tokens) if mode == "prompt" else (args.batch, args.context)
+        per = -(-ctx // page)
+        pool = (torch.randn(n_entries * per, 2 * k * page * d, device="cuda") * 0.5).to(torch.bfloat16)
+        keys, values = (part.unflatten(1, (k, page, d)) for part in pool.chunk(2, dim=1))
+        table = torch.randperm(n_entries * per, device="cuda", dtype=torch.int32).view(n_entries, per).contiguous()
+        n = ctx if mode == "prompt" else n_entries
+        q = torch.randn(n, h * d, device="cuda").to(torch.bfloat16)
+        proj = torch.randn(n, (2 * h + k) * d, device="cuda").to(torch.bfloat16)
+        gate = proj[:, (h + k) * d:]
+        out = torch.empty(n, h * d, dtype=torch.bfloat16, device="cuda")
+        if mode == "prompt":
+            q_start, kv_start, slots, max_q, positions = i32([0, n]), i32([0]), i32([0]), n, i32(list(range(n)))
+            flops, moved = 2 * h * 2 * d * sum(seen(p) for p in range(ctx)), None
+        else:
+            q_start, kv_start, slots, max_q = i32(list(range(n + 1))), i32([ctx - 1] * n), i32(list(range(n))), 1
+            positions = kv_start
+            flops, moved = None, n * seen(ctx - 1) * k * 2 * d * 2
+        tried = [None] if mode == "prompt" or args.splits is None else args.splits
+        for splits in tried:
+            fn = lambda: ops.pooled_window_attention(q, out, q_start, kv_start, slots, keys, values, table, None, None, None, n_entries, max_q,
+                                                     h, k, window=window, keep=keep, pool=0, scale=0.09, sink=sink, gate=gate,
+                                                     max_kv_len=ctx if max_q == 1 else 0, splits=splits)
+            extra = {} if splits is None else {"splits": splits}
+            report(f"kept_window_attention[{mode}]", timer(fn), flops=flops, bytes_moved=moved, entries=n_entries, context=ctx, heads=h,
+                   kv_heads=k, head_dim=d, window=window, keep=keep, **extra)
+        state = torch.zeros(n_entries, (taps - 1) * (h + k) * d, device="cuda")
+        fn = lambda: ops.conv_norm_append(proj, 0, h * d, q, keys, values, conv[0], conv[1], positions, table, q_start, slots, n_entries, max_q,
+                                          h, k, d, freq=freq, q_weight=gain[0], k_weight=gain[1], state=state)
+        report(f"conv_norm_append[{mode}]", timer(fn), bytes_moved=n * (2 * h + 3 * k) * d * 2 + n_entries * state.shape[1] * 8, tokens=n,
+               heads=h, kv_heads=k, head_dim=d, taps=taps)
+
+
+def run_matrix_memory(args) -> None:
+    """The matrix memory on a prompt of --tokens (flops: scores, weighted values, the starting state's part and the state's sum per
+    chunk, each counted once) and on --batch single tokens (bytes: every head's state read and written once), with the gate rows, the
+    norm per head and the output gate."""
+    from torchinferno_b200.kernels.gemm import LinearWeight, linear
+    h, d, v, w = args.heads, args.key_dim, args.value_dim, args.hidden
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device="cuda")
+    timer = Timer(args.iters)
+    gate_w, gate_b, gain = torch.randn(2 * h, w, device="cuda") * w ** -0.5, torch.zeros(2 * h, device="cuda"), torch.ones(h * v, device="cuda")
+    for mode in ("prompt", "single tokens"):
+        n_entries, n = (1, args.tokens) if mode == "prompt" else (args.batch, args.batch)
+        proj = torch.randn(n, 2 * h * (d + v), device="cuda").to(torch.bfloat16)
+        x = torch.randn(n, w, device="cuda").to(torch.bfloat16)
+        out = torch.empty(n, h * v, dtype=torch.bfloat16, device="cuda")
+        state = torch.zeros(n_entries, ops.matrix_memory_state_floats(h, d, v), device="cuda")
+        q_start = i32([0, n]) if mode == "prompt" else i32(list(range(n + 1)))
+        slots, max_q = i32(list(range(n_entries))), (n if mode == "prompt" else 1)
+        fn = lambda: ops.matrix_memory(proj, 0, h * d, 2 * h * d, 2 * h * d + h * v, x, gate_w, gate_b, 15.0, state, q_start, slots, n_entries,
+                                       max_q, gain, 1e-6, out, heads=h, dim=d, vdim=v, q_scale=d ** -0.5)
+        if mode == "prompt":
+            logits = torch.zeros(n, 2 * h, device="cuda")
+            report("matrix_memory[prompt]", timer(fn), flops=2 * h * n * (32 * (d + v) + 2 * d * v), tokens=n, heads=h, key_dim=d, value_dim=v)
+            report("matrix_memory[prompt, gate rows given]", timer(lambda: ops.matrix_memory(
+                proj, 0, h * d, 2 * h * d, 2 * h * d + h * v, x, gate_w, gate_b, 15.0, state, q_start, slots, n_entries, max_q, gain, 1e-6, out,
+                heads=h, dim=d, vdim=v, q_scale=d ** -0.5, logits=logits)), flops=2 * h * n * (32 * (d + v) + 2 * d * v), tokens=n, heads=h)
+            rows = LinearWeight(gate_w.to(torch.bfloat16), few_rows_tcgen05=False)
+            report("gate rows by the library[prompt]", timer(lambda: linear(x, rows, out_dtype=torch.float32)), bytes_moved=n * (w * 2 + h * 8), tokens=n)
+            report("gate rows alone[prompt]", timer(lambda: ops.router_logits(x, gate_w, logits)), bytes_moved=n * (w * 2 + h * 8), tokens=n)
+        else:
+            report("matrix_memory[single tokens]", timer(fn), bytes_moved=2 * n * state.shape[1] * 4, batch=n, heads=h, key_dim=d, value_dim=v)
+
+
+def run_norm_back(args) -> None:
+    """The norm of a sublayer's output with the sum into the residual and the rows in the activation type (bytes: output read,
+    residual read and written, rows written), beside the norm ahead of a sublayer with the residual sum."""
+    w = args.hidden
+    timer = Timer(args.iters)
+    weight = torch.ones(w, device="cuda")
+    for rows in (args.rows, args.batch):
+        y, out = (torch.randn(rows, w, device="cuda").to(torch.bfloat16) for _ in range(2))
+        residual = torch.randn(rows, w, device="cuda")
+        report("unit_norm_add", timer(lambda: ops.unit_norm_add(residual, y, weight, 1e-6, 0.7, out)), bytes_moved=rows * w * 12, rows=rows, hidden=w)
+        report("add_rmsnorm", timer(lambda: ops.add_rmsnorm(y, residual, weight, 1e-6, out)), bytes_moved=rows * w * 12, rows=rows, hidden=w)
+
+
 def run_hyper_streams(args) -> None:
     """A residual in --streams streams: the write of a sublayer's output and the read for the next with the tanh norm in one
     launch (bytes: every stream read and written in fp32, the output rows read, the normed rows written), the read alone,
@@ -792,6 +888,35 @@ def main(argv=None) -> int:
     p.add_argument("--taps", type=int, default=4)
     p.add_argument("--iters", type=int, default=10)
     p.set_defaults(func=run_input_conv)
+    p = sub.add_parser("kept-window-attention")
+    p.add_argument("--tokens", type=int, default=2048)
+    p.add_argument("--batch", type=int, default=8)
+    p.add_argument("--context", type=int, default=2048)
+    p.add_argument("--heads", type=int, default=16)
+    p.add_argument("--kv-heads", type=int, default=8)
+    p.add_argument("--head-dim", type=int, default=128)
+    p.add_argument("--window", type=int, default=512)
+    p.add_argument("--keep", type=int, default=16)
+    p.add_argument("--taps", type=int, default=4)
+    p.add_argument("--splits", type=int, nargs="*", default=None, help="try these numbers of blocks per context of a single token")
+    p.add_argument("--page-size", type=int, default=16)
+    p.add_argument("--iters", type=int, default=10)
+    p.set_defaults(func=run_kept_window_attention)
+    p = sub.add_parser("matrix-memory")
+    p.add_argument("--tokens", type=int, default=2048)
+    p.add_argument("--batch", type=int, default=8)
+    p.add_argument("--heads", type=int, default=16)
+    p.add_argument("--key-dim", type=int, default=128)
+    p.add_argument("--value-dim", type=int, default=128)
+    p.add_argument("--hidden", type=int, default=2048)
+    p.add_argument("--iters", type=int, default=10)
+    p.set_defaults(func=run_matrix_memory)
+    p = sub.add_parser("norm-back")
+    p.add_argument("--rows", type=int, default=2048)
+    p.add_argument("--batch", type=int, default=8)
+    p.add_argument("--hidden", type=int, default=2048)
+    p.add_argument("--iters", type=int, default=10)
+    p.set_defaults(func=run_norm_back)
     p = sub.add_parser("hyper-streams")
     p.add_argument("--rows", type=int, default=2048)
     p.add_argument("--hidden", type=int, default=2048)

@@ -199,19 +199,152 @@ __global__ void __launch_bounds__(kCnaThreads) conv_norm_append_kernel(const T* 
   }
 }
 
+// The same for bf16 rows of at most 8 * 1024 columns and at most four taps: a thread owns eight channels, keeps their taps in
+// registers and slides over kCnaSegment tokens, whose rows it asks for together; the segment's sums of squares are one reduction.
+// grid (segments, entries, 2).  The block of an entry's first segment alone touches the carried rows (a segment is no shorter than
+// what is carried): it reads them first and then leaves the new ones.
+constexpr int kCnaSegment = 4, kCnaFewTaps = 4;
+
+template <int THREADS>
+__global__ void __launch_bounds__(THREADS) conv_norm_append_rows_kernel(const __nv_bfloat16* __restrict__ proj, __nv_bfloat16* __restrict__ q_out, CnaArgs a) {
+  extern __shared__ __align__(16) float sm[];                // cos, then sin: [segment][n_freq] each
+  __shared__ float sums_s[kCnaSegment][33];
+  constexpr int SEG = kCnaSegment, BACK = kCnaFewTaps - 1;
+  const bool is_q = blockIdx.z == 0;
+  const int width = (is_q ? a.heads : a.kv_heads) * a.dim, carried = a.taps - 1;
+  const int channels = (a.heads + a.kv_heads) * a.dim, chan0 = is_q ? 0 : a.heads * a.dim;
+  const int e = threadIdx.x * 8, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+  const bool active = e < width;
+  const float* conv = is_q ? a.q_conv : a.k_conv;
+  const float* weight = is_q ? a.q_weight : a.k_weight;
+  const int entry = blockIdx.y;
+  const int row0 = a.q_start[entry], len = a.q_start[entry + 1] - row0, r0 = blockIdx.x * SEG;
+  // taps and gains do not depend on the kernel before.  w[j] is the tap of the row BACK - j places back (zero where there is none)
+  float w[kCnaFewTaps][8], gain[8];
+#pragma unroll
+  for (int j = 0; j < kCnaFewTaps; ++j) {
+    const int tap = j - (BACK - carried);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) w[j][i] = 0.f;
+    if (active && tap >= 0) cna_load_f32<8>(conv + (size_t)tap * width + e, w[j]);
+  }
+  if (active && weight) cna_load_f32<8>(weight + e, gain);
+  pdl_wait();
+  pdl_trigger();
+  if (r0 >= len) return;
+  const int n = min(SEG, len - r0);
+  const int slot = a.slots[entry];
+  float* state = a.state ? a.state + (size_t)slot * a.state_stride + a.state_off + chan0 : nullptr;
+  const __nv_bfloat16* src = proj + (size_t)row0 * a.ld + (is_q ? a.q_off : a.k_off);
+  float v[SEG][8], ss[SEG];
+#pragma unroll
+  for (int t = 0; t < SEG; ++t) {
+    ss[t] = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[t][i] = 0.f;
+  }
+  if (active) {
+    uint4 raw[SEG + BACK];
+#pragma unroll
+    for (int x = 0; x < SEG + BACK; ++x) {
+      const int r = r0 - BACK + x;
+      raw[x] = r >= 0 && r < r0 + n ? *reinterpret_cast<const uint4*>(src + (size_t)r * a.ld + e) : make_uint4(0, 0, 0, 0);
+    }
+#pragma unroll
+    for (int x = 0; x < SEG + BACK; ++x) {
+      const int r = r0 - BACK + x;
+      float u[8];
+      const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&raw[x]);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float2 f = bf16x2_floats(b[i]);
+        u[2 * i] = f.x;
+        u[2 * i + 1] = f.y;
+      }
+      if (r < 0 && r + carried >= 0) cna_load_f32<8>(state + (size_t)(r + carried) * channels + e, u);      // (r < 0 in the first segment only)
+#pragma unroll
+      for (int t = 0; t < SEG; ++t) {
+        const int j = x - t;                               // this row's place among the taps of token t
+        if (j < 0 || j > BACK) continue;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[t][i] = fmaf(w[j][i], u[i], v[t][i]);
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < SEG; ++t)
+#pragma unroll
+      for (int i = 0; i < 8; ++i) ss[t] = fmaf(v[t][i], v[t][i], ss[t]);
+    if (r0 == 0 && carried > 0)       // what the next step finds: the last projected rows (rows move up in place, a channel by one thread)
+      for (int k = 0; k < carried; ++k) {
+        const int from = len - carried + k;
+        float u[8];
+        if (from >= 0) cna_load<__nv_bfloat16, 8>(src + (size_t)from * a.ld + e, u);
+        else cna_load_f32<8>(state + (size_t)(k + len) * channels + e, u);
+        cna_store_f32<8>(state + (size_t)k * channels + e, u);
+      }
+  }
+  for (int i = threadIdx.x; i < n * a.n_freq; i += blockDim.x) {
+    const int t = i / a.n_freq, f = i - t * a.n_freq;
+    const float angle = (float)a.positions[row0 + r0 + t] * a.freq[f];
+    sm[i] = cosf(angle);
+    sm[SEG * a.n_freq + i] = sinf(angle);
+  }
+#pragma unroll
+  for (int t = 0; t < SEG; ++t) {
+    const float s = warp_sum(ss[t]);
+    if (lane == 0) sums_s[t][warp] = s;
+  }
+  __syncthreads();
+  if (!active) return;
+  const int head = e / a.dim, d = e - head * a.dim;
+  const int* table = a.block_table + (size_t)slot * a.table_stride;
+#pragma unroll
+  for (int t = 0; t < SEG; ++t) {
+    if (t >= n) break;
+    const size_t token = (size_t)row0 + r0 + t;
+    __nv_bfloat16* dst = q_out + token * width + e;
+    if (!is_q) {
+      const int pos = a.positions[token], page = table[pos / a.page_size];
+      if (page < 0 || page >= a.num_pages) {
+        if (a.error_word && threadIdx.x == 0) atomicExch(a.error_word, 0x30000 + (int)(token & 0xffff));
+        continue;
+      }
+      const size_t at = (size_t)page * a.page_stride + ((size_t)head * a.page_size + pos % a.page_size) * a.dim + d;
+      cna_store<__nv_bfloat16, 8>(reinterpret_cast<__nv_bfloat16*>(a.values) + at, v[t]);
+      dst = reinterpret_cast<__nv_bfloat16*>(a.keys) + at;
+    }
+    if (weight) {
+      float total = 0.f;
+      for (int x = 0; x < warps; ++x) total += sums_s[t][x];
+      const float inv = 1.f / sqrtf(total / (float)width + a.eps);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) v[t][i] = v[t][i] * inv * gain[i];
+    }
+#pragma unroll
+    for (int i = 0; i < 8; i += 2) {
+      const int pair = (d + i) >> 1;
+      if (pair >= a.n_freq) continue;
+      const float lo = v[t][i], hi = v[t][i + 1], c = sm[t * a.n_freq + pair], sn = sm[(SEG + t) * a.n_freq + pair];
+      v[t][i] = rope_lo(lo, hi, c, sn);
+      v[t][i + 1] = rope_hi(lo, hi, c, sn);
+    }
+    cna_store<__nv_bfloat16, 8>(dst, v[t]);
+  }
+}
+
 }  // namespace tib
 
 using namespace tib;
 
 // proj: [n_tokens, ld] rows with q at q_off and k at k_off; q_out: [n_tokens, heads * dim]; k_pages / v_pages: first key / value
-// of this layer's first page (heads of `dim` elements in both); state (null when taps is 1): see CnaArgs.
+// of this layer's first page (heads of `dim` elements in both); state (null when taps is 1): see CnaArgs.  max_q_len: the longest entry of the step.
 TIB_API int tib_conv_norm_append(const void* proj, int64_t ld, int q_off, int k_off, const float* q_conv, const float* k_conv, int taps,
                                  const float* q_weight, const float* k_weight, float eps, const float* freq, int n_freq, void* q_out,
                                  void* k_pages, void* v_pages, const int* positions, const int* block_table,
                                  int table_stride, const int* q_start, const int* slots, int n_entries, float* state,
-                                 int64_t state_stride, int64_t state_off, int n_tokens, int heads, int kv_heads, int dim,
-                                 int page_size, int64_t page_stride, int num_pages, int* error_word, int dtype, cudaStream_t stream) {
-  if (n_tokens == 0 || n_entries == 0) return TIB_OK;
+                                 int64_t state_stride, int64_t state_off, int n_tokens, int max_q_len, int heads, int kv_heads,
+                                 int dim, int page_size, int64_t page_stride, int num_pages, int* error_word, int dtype, cudaStream_t stream) {
+  if (n_tokens == 0 || n_entries == 0 || max_q_len == 0) return TIB_OK;
   if (!proj || !q_out || !k_pages || !v_pages || !q_conv || !k_conv || !positions || !block_table || !q_start || !slots) return TIB_E_ARG;
   if ((!q_weight) != (!k_weight) || (n_freq > 0 && !freq) || (taps > 1 && !state)) return TIB_E_ARG;
   if (heads < 1 || kv_heads < 1 || dim < 1 || taps < 1 || n_freq < 0 || 2 * n_freq > dim || page_size < 1) return TIB_E_SIZE;
@@ -237,6 +370,19 @@ TIB_API int tib_conv_norm_append(const void* proj, int64_t ld, int q_off, int k_
     }                                                                                                                \
     TIB_LAUNCH_DEPENDENT(kern, dim3(n_tokens, 2), kCnaThreads, smem, stream, (const T*)proj, (T*)q_out, a);          \
   } while (0)
+  const int wide = (heads > kv_heads ? heads : kv_heads) * dim, segments = ceil_div(max_q_len, kCnaSegment);
+  if (pieces && taps <= kCnaFewTaps && wide <= 8 * 1024 && n_entries <= 65535) {
+    const int threads = ceil_div(wide / 8, 32) * 32;
+    const size_t angles = sizeof(float) * 2 * kCnaSegment * (size_t)n_freq;
+    if (angles <= 48 * 1024) {
+      const dim3 grid(segments, n_entries, 2);
+      if (threads <= 512)
+        TIB_LAUNCH_DEPENDENT(conv_norm_append_rows_kernel<512>, grid, threads, angles, stream, (const __nv_bfloat16*)proj, (__nv_bfloat16*)q_out, a);
+      else
+        TIB_LAUNCH_DEPENDENT(conv_norm_append_rows_kernel<1024>, grid, threads, angles, stream, (const __nv_bfloat16*)proj, (__nv_bfloat16*)q_out, a);
+      return TIB_OK;
+    }
+  }
   if (pieces) TIB_CNA(__nv_bfloat16, 8);
   else if (dtype == TIB_BF16) TIB_CNA(__nv_bfloat16, 1);
   else if (dtype == TIB_F32) TIB_CNA(float, 1);

@@ -37,7 +37,7 @@ constexpr int kMemMaxDim = 512;
 struct MemArgs {
   const void* proj; int64_t ld; int q_off, k_off, v_off, g_off;     // rows of the fused projection (type T); g: the output gate
   float q_scale;
-  const float* logits;                                               // [tokens, 2 * heads] raw gate rows (i of every head, then f), or null:
+  const float* logits; int64_t ld_logits;                            // [tokens, >= 2 * heads] raw gate rows (i of every head, then f), or null:
   const void* x; int64_t ldx; const float* gate_w; int width;       //   the layer's input rows (type T) and the rows' weights [2 * heads, width]
   const float* gate_bias; float cap;                                 // [2 * heads]
   float* state; int64_t state_stride;
@@ -118,7 +118,7 @@ __global__ void __launch_bounds__(kWalkThreads) mem_walk_kernel(MemArgs a) {
     if (tid < cols) v_s[tid] = to_f32(row[a.v_off + h * V + c0 + tid]);
     else if (tid < kMemTile) v_s[tid] = 0.f;
     if (a.logits) {
-      if (tid < 2) gate_s[tid] = a.logits[token * 2 * H + tid * H + h];
+      if (tid < 2) gate_s[tid] = a.logits[token * a.ld_logits + tid * H + h];
     } else {
       // the two gate rows times this token's input
       const T* x = reinterpret_cast<const T*>(a.x) + token * a.ldx;
@@ -238,7 +238,7 @@ __global__ void __launch_bounds__(kGateThreads) mem_gates_kernel(MemArgs a) {
     MemSpan mine = {0.0, -1e300};            // (a thread without a token changes nothing)
     float in = 0.f;
     if (t < len) {
-      const float* z = a.logits + (size_t)(row0 + t) * 2 * H + h;
+      const float* z = a.logits + (size_t)(row0 + t) * a.ld_logits + h;
       in = mem_capped(z[0] + bias_i, a.cap);
       const double f = (double)mem_log_sigmoid(mem_capped(z[H] + bias_f, a.cap));
       mine = {f, (double)in - f};
@@ -715,13 +715,13 @@ TIB_API int tib_matrix_memory_max_dim() { return kMemMaxDim; }
 TIB_API int tib_matrix_memory_takes_chunks(int dim, int vdim) { return dim % 8 == 0 && vdim % 8 == 0 && dim <= 256; }
 
 // proj: rows of `dtype` with q, k, v and the output gate's logits at their offsets; logits [n_tokens, 2 * heads] fp32 (raw gate
-// rows), or null and x / gate_w [2 * heads, width]; gate_bias [2 * heads]; state: per slot (stride state_stride floats, a
+// rows, ld_logits apart), or null and x / gate_w [2 * heads, width]; gate_bias [2 * heads]; state: per slot (stride state_stride floats, a
 // multiple of 4) heads * D * V + heads * ceil(V / tile) * (D + 1) floats.  norm_weight [heads * V] (V at most a tile): out gets
 // the normed and gated rows in `dtype`; null: y gets fp32 rows.  chunks != 0: the chunk form (bf16, logits given), with cum
 // [heads, n_tokens] double, log_in and top [heads, n_tokens], top0 [heads, n_entries], run_state [run_capacity, heads, D, V],
 // run_n [run_capacity, heads, D], run_keep [run_capacity, heads]; run_capacity >= n_tokens / chunk + n_entries.
 TIB_API int tib_matrix_memory(const void* proj, int64_t ld, int q_off, int k_off, int v_off, int g_off, float q_scale,
-                              const float* logits, const void* x, int64_t ldx, const float* gate_w, int width,
+                              const float* logits, int64_t ld_logits, const void* x, int64_t ldx, const float* gate_w, int width,
                               const float* gate_bias, float cap, float* state, int64_t state_stride, const int* q_start,
                               const int* slots, const float* norm_weight, float eps, float* y, void* out, int heads, int D, int V,
                               int n_entries, int n_tokens, int max_q_len, int chunks, double* cum, float* log_in, float* top,
@@ -730,11 +730,12 @@ TIB_API int tib_matrix_memory(const void* proj, int64_t ld, int q_off, int k_off
   if (n_entries == 0 || n_tokens == 0 || max_q_len == 0) return TIB_OK;
   if (!proj || !gate_bias || !state || !q_start || !slots || (!y && !out) || (norm_weight && !out) || (!norm_weight && !y)) return TIB_E_ARG;
   if (!logits && (!x || !gate_w || width < 1)) return TIB_E_ARG;
+  if (logits && ld_logits < 2 * (int64_t)heads) return TIB_E_SIZE;
   if (heads < 1 || D < 1 || D > kMemMaxDim || V < 1 || !(cap > 0.f) || n_entries > 65535 || state_stride % 4) return TIB_E_SIZE;
   if (dtype != TIB_F32 && dtype != TIB_BF16) return TIB_E_DTYPE;
   MemArgs a = {};
   a.proj = proj; a.ld = ld; a.q_off = q_off; a.k_off = k_off; a.v_off = v_off; a.g_off = g_off; a.q_scale = q_scale;
-  a.logits = logits; a.x = x; a.ldx = ldx; a.gate_w = gate_w; a.width = width; a.gate_bias = gate_bias; a.cap = cap;
+  a.logits = logits; a.ld_logits = ld_logits; a.x = x; a.ldx = ldx; a.gate_w = gate_w; a.width = width; a.gate_bias = gate_bias; a.cap = cap;
   a.state = state; a.state_stride = state_stride; a.q_start = q_start; a.slots = slots; a.norm_weight = norm_weight; a.eps = eps;
   a.y = y; a.out = out; a.heads = heads; a.D = D; a.V = V; a.tiles = ceil_div(V, kMemTile); a.n_tokens = n_tokens;
   a.cum = cum; a.log_in = log_in; a.top = top; a.top0 = top0; a.run_state = run_state; a.run_n = run_n; a.run_keep = run_keep;

@@ -1720,7 +1720,7 @@ def talking_heads_attention(q: torch.Tensor, out: torch.Tensor, q_start: torch.T
 # Queries and keys that pass a short convolution ahead of norm and rotation (csrc/conv_norm_append.cu).
 def conv_norm_append(proj: torch.Tensor, q_off: int, k_off: int, q_out: torch.Tensor, keys: torch.Tensor, values: torch.Tensor,
                      q_conv: torch.Tensor, k_conv: torch.Tensor, positions: torch.Tensor, block_table: torch.Tensor,
-                     q_start: torch.Tensor, slots: torch.Tensor, n_entries: int, heads: int, kv_heads: int, dim: int, *,
+                     q_start: torch.Tensor, slots: torch.Tensor, n_entries: int, max_q_len: int, heads: int, kv_heads: int, dim: int, *,
                      freq: torch.Tensor, q_weight: torch.Tensor | None = None, k_weight: torch.Tensor | None = None, eps: float = 1e-6,
                      state: torch.Tensor | None = None, state_off: int = 0, error_word: torch.Tensor | None = None) -> torch.Tensor:
     """Per channel of the q and k columns of ``proj``, y_t = sum_j conv[j] * u_(t - taps + 1 + j) within each entry (``q_conv`` /
@@ -1758,7 +1758,7 @@ def conv_norm_append(proj: torch.Tensor, q_off: int, k_off: int, q_out: torch.Te
         _ptr(proj), c_int64(proj.stride(0)), c_int(q_off), c_int(k_off), _ptr(q_conv), _ptr(k_conv), c_int(taps), _ptr(q_weight),
         _ptr(k_weight), c_float(eps), _ptr(freq), c_int(freq.numel()), _ptr(q_out), _ptr(keys), _ptr(values), _ptr(positions),
         _ptr(block_table), c_int(block_table.stride(0)), _ptr(q_start), _ptr(slots), c_int(n_entries), _ptr(state if taps > 1 else None),
-        c_int64(stride), c_int64(state_off), c_int(n), c_int(heads), c_int(kv_heads), c_int(dim), c_int(page_size),
+        c_int64(stride), c_int64(state_off), c_int(n), c_int(max_q_len), c_int(heads), c_int(kv_heads), c_int(dim), c_int(page_size),
         c_int64(page_stride), c_int(num_pages), _ptr(error_word), c_int(_code(proj.dtype)), _stream()))
     return q_out
 
@@ -1783,12 +1783,13 @@ def matrix_memory_state_floats(heads: int, dim: int, vdim: int) -> int:
 def matrix_memory(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off: int, x: torch.Tensor, gate_weight: torch.Tensor,
                   gate_bias: torch.Tensor, cap: float, state: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, n_entries: int,
                   max_q_len: int, norm_weight: torch.Tensor, eps: float, out: torch.Tensor, *, heads: int, dim: int, vdim: int,
-                  q_scale: float, walk: bool | None = None) -> torch.Tensor:
+                  q_scale: float, walk: bool | None = None, logits: torch.Tensor | None = None) -> torch.Tensor:
     """Per head, with i = cap tanh((w_i . x + b_i) / cap), f = logsigmoid(cap tanh((w_f . x + b_f) / cap)) and m_t = max(f + m, i):
     S_t = exp(f + m - m_t) S + exp(i - m_t) k v^T, n_t likewise with k alone, y = S_t^T q / (max(|n_t . q|, exp(-m_t)) + 1e-6);
     out = y / rms(y) * norm_weight * sigmoid(gate).  ``proj`` holds q, k, v and the gate's logits at their columns (q is multiplied by
     ``q_scale``); ``gate_weight`` [2 * heads, width] (i of every head, then f) and ``gate_bias`` are fp32, ``x`` the input rows they
-    multiply; ``state`` [slots, floats] is read and left updated.  ``walk``: token by token (None: decided by the portions' length
+    multiply (``logits`` [tokens, >= 2 * heads] fp32: the rows' products, if the caller has them); ``state`` [slots, floats] is read and
+    left updated.  ``walk``: token by token (None: decided by the portions' length
     and the shapes)."""
     _rows_of(proj, "proj"), _rows_of(x, "x"), _need(state, "state", torch.float32), _need(out, "out", proj.dtype)
     for name, t in (("gate_weight", gate_weight), ("gate_bias", gate_bias), ("norm_weight", norm_weight)):
@@ -1807,8 +1808,11 @@ def matrix_memory(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off:
         raise KernelError("matrix_memory: entry arrays are shorter than n_entries")
     takes_chunks = proj.dtype == torch.bfloat16 and bool(library.tib_matrix_memory_takes_chunks(c_int(dim), c_int(vdim)))
     chunks = takes_chunks and max_q_len > MATRIX_MEMORY_WALK if walk is None else not walk
-    logits = None
-    if max_q_len > 1:      # (a step of single tokens works its gate rows out in the same launch)
+    if logits is not None:
+        _rows_of(logits, "logits")
+        if logits.dtype != torch.float32 or logits.shape[0] != n or logits.shape[1] < 2 * heads:
+            raise KernelError("matrix_memory: the gate rows' products do not fit")
+    elif max_q_len > 1:      # (a step of single tokens works its gate rows out in the same launch)
         logits = router_logits(x, gate_weight, torch.empty((n, 2 * heads), dtype=torch.float32, device=dev))
     fused = vdim <= MATRIX_MEMORY_TILE
     y = None if fused else torch.empty((n, heads * vdim), dtype=torch.float32, device=dev)
@@ -1825,7 +1829,7 @@ def matrix_memory(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, g_off:
         count_launches(3)
     _check("matrix_memory", library.tib_matrix_memory(
         _ptr(proj), c_int64(proj.stride(0)), c_int(q_off), c_int(k_off), c_int(v_off), c_int(g_off), c_float(q_scale), _ptr(logits),
-        _ptr(x), c_int64(x.stride(0)), _ptr(gate_weight), c_int(x.shape[1]), _ptr(gate_bias), c_float(cap), _ptr(state),
+        c_int64(logits.stride(0) if logits is not None else 0), _ptr(x), c_int64(x.stride(0)), _ptr(gate_weight), c_int(x.shape[1]), _ptr(gate_bias), c_float(cap), _ptr(state),
         c_int64(state.stride(0)), _ptr(q_start), _ptr(slots), _ptr(norm_weight if fused else None), c_float(eps), _ptr(y),
         _ptr(out if fused else None), c_int(heads), c_int(dim), c_int(vdim), c_int(n_entries), c_int(n), c_int(max_q_len),
         c_int(int(chunks)), _ptr(cum), _ptr(log_in), _ptr(top), _ptr(top0), _ptr(run_state), _ptr(run_n), _ptr(run_keep),

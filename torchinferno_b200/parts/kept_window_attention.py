@@ -115,7 +115,7 @@ class KeptWindowAttention(Mixer):
         proj = linear(x, self.in_weight)                                    # [q | k | gate]
         q = torch.empty((n, h * d), dtype=x.dtype, device=x.device)
         ops.conv_norm_append(proj, 0, self.k_off, q, kv.keys, kv.values, self.q_conv, self.k_conv, batch.positions, kv.block_table,
-                             batch.q_start, batch.slots, batch.n_entries, h, g, d, freq=self.position.rotary_table()[0],
+                             batch.q_start, batch.slots, batch.n_entries, batch.max_q_len, h, g, d, freq=self.position.rotary_table()[0],
                              q_weight=self.q_norm_weight, k_weight=self.k_norm_weight, eps=self.row_norm_eps or 0.0,
                              state=ctx.state, error_word=ctx.error_word)
         out = torch.empty((n, h * d), dtype=x.dtype, device=x.device)

@@ -10,7 +10,7 @@ i = cap tanh((w_i . x + b_i) / cap) and a log forget gate f = logsigmoid(cap tan
 Each head's o is divided by its root mean square (``eps``); the heads side by side are multiplied by a weight (``norm``) and by
 sigmoid(W_g x), then projected by W_o.  S, n and m live in 32-bit in the cache manager's state slots (zero for a new request) and are
 carried from step to step; the mixer keeps no keys.  q, k, v and the gate's logits are one product; the two gate rows per head are
-multiplied in fp32 in either mode.  The kernels (csrc/matrix_memory.cu) take the step's whole ragged batch, prompt portions and
+summed in fp32 and stay fp32 in either mode (on long portions in bfloat16 by a product with fp32 output).  The kernels (csrc/matrix_memory.cu) take the step's whole ragged batch, prompt portions and
 single tokens alike, and read it through its device arrays only.
 """
 from __future__ import annotations
@@ -22,6 +22,13 @@ import torch
 from torchinferno_b200.kernels import ops
 from torchinferno_b200.kernels.gemm import LinearWeight, linear
 from torchinferno_b200.parts.base import LayerContext, Mixer, StateSpec, WeightSpec, register_part
+
+
+MANY_ROWS = 128        # from this many rows on the gate rows are a library product
+
+
+def up_to_eight(n: int) -> int:
+    return (n + 7) // 8 * 8
 
 
 class MatrixMemory(Mixer):
@@ -37,16 +44,14 @@ class MatrixMemory(Mixer):
         self.gate_cap, self.eps = float(gate_cap), float(eps)
         self.names = {"q": q_name, "k": k_name, "v": v_name, "g": g_name, "o": o_name, "norm": norm_name, "i": i_name, "f": f_name,
                       "ib": i_name + bias_suffix, "fb": f_name + bias_suffix}
-
-        def up(at: int) -> int:      # (every part of the product starts on a 16-byte boundary in bfloat16)
-            return (at + 7) // 8 * 8
-        self.k_off = up(heads * dim)
-        self.v_off = up(self.k_off + heads * dim)
-        self.g_off = up(self.v_off + heads * value_dim)
-        self.in_width = up(self.g_off + heads * value_dim)
+        # (every part of the product starts on a 16-byte boundary in bfloat16)
+        self.k_off = up_to_eight(heads * dim)
+        self.v_off = up_to_eight(self.k_off + heads * dim)
+        self.g_off = up_to_eight(self.v_off + heads * value_dim)
+        self.in_width = up_to_eight(self.g_off + heads * value_dim)
         self.in_weight: LinearWeight | None = None
         self.o_weight: LinearWeight | None = None
-        self.gate_weight = self.gate_bias = self.norm_weight = None
+        self.gate_weight = self.gate_bias = self.norm_weight = self.gate_rows = None
 
     def weight_specs(self) -> list[WeightSpec]:
         n, w, qk, vv = self.names, self.hidden_size, self.heads * self.dim, self.heads * self.value_dim
@@ -66,6 +71,10 @@ class MatrixMemory(Mixer):
             rows[at:at + part.shape[0]] = part
         self.in_weight = LinearWeight(rows, few_rows_tcgen05=None)
         self.o_weight = LinearWeight(weights[n["o"]], few_rows_tcgen05=None)
+        if self.dtype == torch.bfloat16 and weights[n["i"]].dtype == weights[n["f"]].dtype == torch.bfloat16:
+            rows = torch.zeros((up_to_eight(2 * self.heads), self.hidden_size), dtype=torch.bfloat16, device=first.device)
+            rows[:self.heads], rows[self.heads:2 * self.heads] = weights[n["i"]], weights[n["f"]]
+            self.gate_rows = LinearWeight(rows, few_rows_tcgen05=False)
         self.gate_weight = torch.cat([weights[n["i"]], weights[n["f"]]], dim=0).to(torch.float32).contiguous()
         self.gate_bias = torch.cat([weights[n["ib"]], weights[n["fb"]]], dim=0).to(torch.float32).contiguous()
         self.norm_weight = weights[n["norm"]].to(torch.float32).contiguous()
@@ -81,9 +90,12 @@ class MatrixMemory(Mixer):
         batch = ctx.batch
         proj = linear(x, self.in_weight)                                    # [q | k | v | gate]
         rows = torch.empty((x.shape[0], self.heads * self.value_dim), dtype=x.dtype, device=x.device)
+        logits = None
+        if self.gate_rows is not None and x.shape[0] >= MANY_ROWS and batch.max_q_len > 1:
+            logits = linear(x, self.gate_rows, out_dtype=torch.float32)
         ops.matrix_memory(proj, 0, self.k_off, self.v_off, self.g_off, x, self.gate_weight, self.gate_bias, self.gate_cap, ctx.state,
                           batch.q_start, batch.slots, batch.n_entries, batch.max_q_len, self.norm_weight, self.eps, rows,
-                          heads=self.heads, dim=self.dim, vdim=self.value_dim, q_scale=self.dim ** -0.5)
+                          heads=self.heads, dim=self.dim, vdim=self.value_dim, q_scale=self.dim ** -0.5, logits=logits)
         return linear(rows, self.o_weight)
 
 
