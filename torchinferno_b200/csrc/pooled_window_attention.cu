@@ -861,13 +861,14 @@ pwa_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __r
 }
 
 // Adds the parts of a context that was shared out over blocks, in the order of the parts: out = sum_s o_s 2^(m_s - top)
-// / (sum_s l_s 2^(m_s - top) + 2^(sink - top)), times the gate.  One block per token, a warp per head.
+// / (sum_s l_s 2^(m_s - top) + 2^(sink - top)), times the gate.  grid (tokens, groups of four heads), a warp per head.
 template <int DV>
 __global__ void __launch_bounds__(128) pwa_merge_kernel(__nv_bfloat16* __restrict__ out, PwaArgs a) {
   pdl_wait();
   pdl_trigger();
   const int token = blockIdx.x, lane = threadIdx.x & 31;
-  for (int head = threadIdx.x >> 5; head < a.heads; head += blockDim.x >> 5) {
+  const int head = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (head < a.heads) {
     float top = -CUDART_INF_F;
     for (int s = 0; s < a.n_splits; ++s)
       top = fmaxf(top, a.partial[(((size_t)s * a.n_tokens + token) * a.heads + head) * (DV + 2)]);
@@ -937,7 +938,7 @@ static int pwa_launch_mma(const void* q, void* out, PwaArgs a, int n_entries, in
       const int status = a.keep > 0 ? pwa_launch_mma_staged<DK, DV, kPmFewRowStages, true, kPwaKeep>(q, out, a, grid, stream)
                                     : pwa_launch_mma_staged<DK, DV, kPmFewRowStages, true, kPwaRel>(q, out, a, grid, stream);
       if (status != TIB_OK) return status;
-      TIB_LAUNCH_DEPENDENT(pwa_merge_kernel<DV>, a.n_tokens, 128, 0, stream, (__nv_bfloat16*)out, a);
+      TIB_LAUNCH_DEPENDENT(pwa_merge_kernel<DV>, dim3(a.n_tokens, ceil_div(a.heads, 4)), 128, 0, stream, (__nv_bfloat16*)out, a);
       return TIB_OK;
     }
     a.n_splits = 1;
